@@ -15,7 +15,7 @@ What is here instead:
   valid for every entry of its group.  A request has one block table per
   group.  A mixer that caches one vector per token (``PagedVectorNeed``: a
   latent that keys and values are derived from) joins a group of its width,
-  window and kept first tokens, whose tensor is ``[entries, pages, page_size, width]``.
+  window, chunk and kept first tokens, whose tensor is ``[entries, pages, page_size, width]``.
 * **Pages on demand.**  ``append`` allocates the pages that the tokens of the
   coming step need, in all groups or in none; ``commit`` advances the
   request's length after the step has run (the reference's two-phase
@@ -177,7 +177,7 @@ class CacheManager:
                                                         dtype=need.state.dtype, device=device)
                 need = need.paged
             if isinstance(need, (PagedKVNeed, PagedVectorNeed)):
-                key = (("vector", need.width, need.window, need.keep_first) if isinstance(need, PagedVectorNeed)
+                key = (("vector", need.width, need.window, need.keep_first, need.chunk) if isinstance(need, PagedVectorNeed)
                        else (need.kv_heads, need.head_dim, need.window))
                 if key not in by_key:
                     by_key[key] = len(self.groups)
@@ -226,9 +226,12 @@ class CacheManager:
 
     def _first_needed_page(self, grp: CacheGroup, length: int) -> int:
         """Index of the first page that a query at position >= ``length`` can still read."""
-        if grp.need.window is None:
-            return 0
-        return max(0, length - grp.need.window + 1) // self.page_size
+        n = grp.need
+        first = 0 if n.window is None else max(0, length - n.window + 1)
+        chunk = getattr(n, "chunk", None)
+        if chunk is not None:
+            first = max(first, length - length % chunk)
+        return first // self.page_size
 
     def pages_needed(self, rid: Hashable, n_new: int) -> List[int]:
         """Pages per group that ``append(rid, n_new)`` would allocate."""

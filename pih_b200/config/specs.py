@@ -87,7 +87,14 @@ class ScalarNormSpec:
 class GatedDeltaSpec:
     """Gated delta rule: a matrix state ``S [key_dim, value_dim]`` per head that decays, is corrected towards the
     new value along the new key, and is read with the query.  q and k have ``kv_heads`` heads shared by groups of
-    value heads; q, k and v pass a short causal convolution and SiLU; q and k are made unit vectors."""
+    value heads; q, k and v pass a short causal convolution and SiLU; q and k are made unit vectors.  Options, each a
+    mechanism of its own:
+
+    * ``decay_per`` "head": one decay a head; "channel": one a head and key channel, which decays that row of S;
+    * ``decay_rank``: the decay logits come through a narrow projection (``decay_down`` then ``decay_up``) instead of
+      one matrix (``decay``);
+    * ``gate_rank``: so does the gate of the read-out (``gate_down``, ``gate_up`` instead of ``gate``);
+    * ``gate_activation`` "silu" or "sigmoid"."""
     hidden: int
     heads: int
     kv_heads: int
@@ -96,10 +103,20 @@ class GatedDeltaSpec:
     conv_taps: int
     norm_eps: float                   # of the per-head RMS norm of the read-out
     unit_eps: float = 1e-6            # inside the root of the unit norm of q and k
+    decay_per: str = "head"
+    decay_rank: Optional[int] = None
+    gate_rank: Optional[int] = None
+    gate_activation: str = "silu"
     kind: str = "gated_delta"
     names: Mapping[str, str] = _names(q="mix.q", k="mix.k", v="mix.v", q_conv="mix.q.conv", k_conv="mix.k.conv",
                                       v_conv="mix.v.conv", beta="mix.b", decay="mix.a", decay_log="mix.A_log",
-                                      decay_bias="mix.dt_bias", out_norm="mix.norm", gate="mix.g", o="mix.o")
+                                      decay_bias="mix.dt_bias", out_norm="mix.norm", gate="mix.g", o="mix.o",
+                              decay_down="mix.a1", decay_up="mix.a2", gate_down="mix.g1", gate_up="mix.g2")
+
+    @property
+    def decays(self) -> int:
+        """Decay logits a row."""
+        return self.heads * (self.key_dim if self.decay_per == "channel" else 1)
 
     @property
     def qk_size(self) -> int:
@@ -108,6 +125,37 @@ class GatedDeltaSpec:
     @property
     def v_size(self) -> int:
         return self.heads * self.value_dim
+
+
+@dataclass(frozen=True)
+class SelectiveScanSpec:
+    """Selective scan: ``inner`` channels of ``state`` numbers each.  Two branches read the block's input; the one passes
+    a short causal convolution (with a bias) and SiLU and drives the recurrence ``S[c, n] <- exp(dt_c A[c, n]) S[c, n] +
+    dt_c x_c B_n``, ``y_c = sum_n S[c, n] C_n + D_c x_c`` with ``A = -exp(A_log)``, whose B, C and (through ``dt_rank``
+    numbers) step sizes ``dt = softplus(.)`` are projections of it; SiLU of the other multiplies the output."""
+    hidden: int
+    inner: int
+    state: int
+    dt_rank: int
+    conv_taps: int
+    kind: str = "selective_scan"
+    names: Mapping[str, str] = _names(w_in="mix.in", conv="mix.conv", conv_bias="mix.conv.b", x="mix.x", dt="mix.dt",
+                                      dt_bias="mix.dt.b", a_log="mix.A_log", skip="mix.D", o="mix.o")
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers side by side that read the same input: ``left_scale * left(x) + right_scale * right(x)``.  The specs'
+    tensor names are below the block's prefix as anywhere.  At most one of the two may ask for a paged cache."""
+    left: object
+    right: object
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind: str = "parallel"
+
+    @property
+    def hidden(self) -> int:
+        return self.left.hidden
 
 
 @dataclass(frozen=True)
@@ -265,7 +313,7 @@ class DiffAttentionSpec:
 class BiasedMLPSpec:
     """Two-matrix feed-forward with biases: ``W_down act(W_up x + b_up) + b_down``.  ``activation`` "xielu": for
     z > 0 ``softplus(p) z^2 + z / 2``, else ``(1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2`` with the two learned
-    numbers (p, q) of the tensor ``act``."""
+    numbers (p, q) of the tensor ``act``; "gelu_erf": ``z / 2 (1 + erf(z / sqrt(2)))``, without a tensor."""
     hidden: int
     intermediate: int
     activation: str = "xielu"
@@ -360,6 +408,8 @@ class WindowAttentionSpec:
       ``bucket(n) = n`` below ``bias_rows // 2`` and beyond it ``min(bias_rows - 1, half + floor(ln(n / half) /
       ln(bias_far / half) * (bias_rows - half)))``;
     * ``softcap``: the scaled score becomes ``softcap * tanh(score / softcap)``;
+    * ``chunk`` > 0: a row sees only the keys of its own chunk of that many places, counted from place 0 of the sequence
+      (``window`` 0 beside it: all of the chunk's keys up to the row);
     * ``head_gate``: head h's output is multiplied by ``sigmoid`` of a one-row projection of the mixer's input."""
     hidden: int
     heads: int
@@ -384,6 +434,7 @@ class WindowAttentionSpec:
     # how many keys back the cache has to reach (another entry that reads this cache may look further back than
     # ``window``); None: ``window``
     cache_window: Optional[int] = None
+    chunk: int = 0
     kind: str = "window_attention"
     names: Mapping[str, str] = _names(q="mix.q", k="mix.k", v="mix.v", o="mix.o", q_norm="mix.q.norm", k_norm="mix.k.norm",
                                       q_conv="mix.q.conv", k_conv="mix.k.conv", v_conv="mix.v.conv", bias="mix.rel",
@@ -418,7 +469,8 @@ class BlockSpec:
     for ``arrangement == "outnorm"`` (the norms sit on the sub-layers' outputs,
     the sub-layers read the stream itself); ``arrangement == "hyper"``: the pre-norm
     layer over several streams (``hyper``); ``ffn`` and ``norm_post`` None: the layer has
-    no feed-forward.  ``prefix`` is the layer's tensor-name prefix in the
+    no feed-forward.  ``residual_scale`` multiplies what a "prenorm" layer's
+    sub-layers add to the stream.  ``prefix`` is the layer's tensor-name prefix in the
     weight files."""
     prefix: str
     mixer: object
@@ -429,15 +481,21 @@ class BlockSpec:
     names: Mapping[str, str] = _names(norm_in="input_layernorm.",
                                       norm_post="post_attention_layernorm.")
     hyper: Optional[HyperSpec] = None
+    residual_scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class ScheduleEntry:
     """Run layer ``layer``.  ``reads_cache_of`` names an earlier entry of the
     schedule (by its index in the list) whose cache this entry's mixer reads
-    instead of keeping one of its own."""
+    instead of keeping one of its own.  Right before the layer, ``add_embedding``
+    adds the model's embedding output to the stream once more, and ``add_vector``
+    a row of the model's table of vectors (``ModelSpec.vectors_name``): what a
+    loop over layers does where a pass begins."""
     layer: int
     reads_cache_of: Optional[int] = None
+    add_embedding: bool = False
+    add_vector: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -475,6 +533,11 @@ class ModelSpec:
     # the logits are the head's product times this number
     logit_scale: float = 1.0
     bigram: Optional[BigramSpec] = None
+    # the embedding output is the table's row times this number (a 32-bit stream)
+    embed_scale: float = 1.0
+    # a table [vectors, hidden] of vectors that schedule entries add to the stream (``ScheduleEntry.add_vector``)
+    vectors_name: Optional[str] = None
+    vectors: int = 0
 
     def validate(self) -> None:
         for i, e in enumerate(self.schedule):
@@ -487,3 +550,16 @@ class ModelSpec:
                 if self.schedule[e.reads_cache_of].reads_cache_of is not None:
                     raise ValueError(f"schedule entry {i} reads the cache of entry {e.reads_cache_of}, "
                                      "which keeps none of its own")
+            if e.add_vector is not None and not (self.vectors_name is not None and 0 <= e.add_vector < self.vectors):
+                raise ValueError(f"schedule entry {i} adds vector {e.add_vector}, the model has {self.vectors}")
+            if (e.add_embedding or e.add_vector is not None) and (
+                    self.stream_dtype != "float32" or self.blocks[e.layer].arrangement != "prenorm"):
+                raise ValueError(f"schedule entry {i}: only a pre-norm layer on a 32-bit stream takes an addition before it")
+            if e.add_embedding and (self.bigram is not None or self.position_name is not None or self.streams):
+                raise ValueError(f"schedule entry {i}: an embedding of several tables cannot be added again")
+        if self.embed_scale != 1.0 and (self.stream_dtype != "float32" or self.bigram is not None
+                                        or self.position_name is not None or self.streams):
+            raise ValueError("a scaled embedding goes with one 32-bit stream and one table")
+        if any(b.residual_scale != 1.0 and (b.arrangement != "prenorm" or self.stream_dtype != "float32")
+               for b in self.blocks):
+            raise ValueError("residual_scale goes with pre-norm layers on a 32-bit stream")

@@ -53,6 +53,12 @@ template <typename T> __device__ __forceinline__ float round_to(float v) {
   return to_float<T>(from_float<T>(v));
 }
 
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
+
+// z / 2 (1 + erf(z / sqrt(2)))
+__device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(0.7071067811865476f * z)); }
+
 // silu(g) * u in 32-bit.  The 32-bit stream uses expf and a true division, as the reference's kernel does
 // (kernels/cuda/qwen_bf16_primitives.cu:274-283); the bf16 stream uses the special-function unit's exp2 and
 // reciprocal, whose two-ulp error in 32-bit is a five-hundredth of a bf16 rounding step.

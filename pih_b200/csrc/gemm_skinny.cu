@@ -87,7 +87,9 @@ struct SkinnyParams {
   long long ldx, ldw, ldo;
   int stages;                                    // of the ring of units
   int activation;                                // of the gated epilogue: 0 SiLU, 1 the tanh form of GELU
-  int unary;                                     // of the plain epilogue: 0 none, 1 the square of max(rounded product, 0)
+  int unary;                                     // of the plain epilogue: 0 none, 1 the square of max(rounded product, 0),
+                                                 // 2 GELU (error-function form) of the rounded product plus the bias
+  const float* bias;                             // [N], with unary 2
   uint32_t* error;
 };
 
@@ -348,6 +350,8 @@ __global__ void __launch_bounds__(SK_THREADS, 2) skinny_gemm_kernel(const Skinny
         if (p.unary == 1) {                                  // the activation of a two-matrix feed-forward, on the product's rounding
           sum = fmaxf(__bfloat162float(__float2bfloat16_rn(sum)), 0.0f);
           sum *= sum;
+        } else if (p.unary == 2) {
+          sum = gelu_erf_f(__bfloat162float(__float2bfloat16_rn(sum)) + p.bias[col]);
         }
         out[etok * p.ldo + col] = from_float<OT>(sum);
       }
@@ -605,12 +609,11 @@ extern "C" int pih_set_skinny_rule(int on) {
 //              output projection, with its two roundings; rows of ldo elements; may not be `out` itself
 //   error      the device's error word (a bounded wait that ran out is reported there)
 // Returns PIH_ERR_UNSUPPORTED for shapes it does not take (the caller uses the separate kernels).
-extern "C" int pih_gemm_skinny(const void* x, const void* delta, void* x_out, int norm_dtype, const void* norm_w,
-                               float eps, const void* W, void* out, const void* residual, int M, int N, int K,
-                               long long ldx, long long ldw, long long ldo, int swiglu, uint32_t* error, void* stream) {
+static int skinny_product(const void* x, const void* delta, void* x_out, int norm_dtype, const void* norm_w, float eps,
+                          const void* W, void* out, const void* residual, int M, int N, int K, long long ldx, long long ldw,
+                          long long ldo, int swiglu, const void* bias, uint32_t* error, void* stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (swiglu < 0 || swiglu > 3) return PIH_ERR_BAD_ARGUMENT;
-  if (!skinny_takes(x, W, M, K, ldx, ldw) || (swiglu && swiglu != 3 && N % 16) || (swiglu && residual != nullptr) ||
+  if (!skinny_takes(x, W, M, K, ldx, ldw) || (swiglu && swiglu < 3 && N % 16) || (swiglu && residual != nullptr) ||
       (reinterpret_cast<uintptr_t>(norm_w) & 15) || residual == out || (norm_w != nullptr && K % 8) ||
       (delta != nullptr && ((reinterpret_cast<uintptr_t>(delta) & 15) || x_out == nullptr || x_out == x)))
     return PIH_ERR_UNSUPPORTED;
@@ -641,13 +644,30 @@ extern "C" int pih_gemm_skinny(const void* x, const void* delta, void* x_out, in
   p.error = error;
   const bool sw = swiglu == 1 || swiglu == 2;
   p.activation = swiglu == 2 ? 1 : 0;
-  p.unary = swiglu == 3 ? 1 : 0;
+  p.unary = swiglu == 3 ? 1 : (swiglu == 4 ? 2 : 0);
+  p.bias = static_cast<const float*>(bias);
 #define PIH_SKINNY(MR, NORM, NW) dispatch_skinny<MR, NORM, NW>(sw, p, s)
   if (norm_w == nullptr) return M <= 8 ? PIH_SKINNY(8, false, float) : PIH_SKINNY(16, false, float);
   if (norm_dtype == PIH_F32) return M <= 8 ? PIH_SKINNY(8, true, float) : PIH_SKINNY(16, true, float);
   if (norm_dtype == PIH_BF16) return M <= 8 ? PIH_SKINNY(8, true, __nv_bfloat16) : PIH_SKINNY(16, true, __nv_bfloat16);
 #undef PIH_SKINNY
   return PIH_ERR_BAD_ARGUMENT;
+}
+
+extern "C" int pih_gemm_skinny(const void* x, const void* delta, void* x_out, int norm_dtype, const void* norm_w,
+                               float eps, const void* W, void* out, const void* residual, int M, int N, int K,
+                               long long ldx, long long ldw, long long ldo, int swiglu, uint32_t* error, void* stream) {
+  if (swiglu < 0 || swiglu > 3) return PIH_ERR_BAD_ARGUMENT;
+  return skinny_product(x, delta, x_out, norm_dtype, norm_w, eps, W, out, residual, M, N, K, ldx, ldw, ldo, swiglu, nullptr,
+                        error, stream);
+}
+
+// out[M, N] = GELU (error-function form) of round(x . W^T) + bias, bias fp32 [N]: the first half of a two-matrix
+// feed-forward with biases.  Shapes as pih_gemm_skinny's.
+extern "C" int pih_gemm_skinny_bias_gelu(const void* x, const void* W, const void* bias, void* out, int M, int N, int K,
+                                         long long ldx, long long ldw, long long ldo, uint32_t* error, void* stream) {
+  if (bias == nullptr) return PIH_ERR_BAD_ARGUMENT;
+  return skinny_product(x, nullptr, nullptr, 0, nullptr, 0.0f, W, out, nullptr, M, N, K, ldx, ldw, ldo, 4, bias, error, stream);
 }
 
 // The same product with 32-bit output and nothing fused: out[M, N] (float) = x[M, K] . W[N, K]^T, for the LM

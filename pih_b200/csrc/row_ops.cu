@@ -7,7 +7,7 @@
 //   rotate_heads    the columns offset .. offset + rot of every head rotated by position * f_i (32-bit angles), the
 //                   pairs being halves (i, i + rot / 2) or neighbours (2i, 2i + 1)
 //   gate_mul        a * sigmoid(g) or a * silu(g), the gate a strided view
-//   unary_act       relu(z)^2
+//   unary_act       relu(z + bias)^2 or the error-function form of GELU of z + bias
 //   scale_rows      x *= s in place (32-bit)
 #include "common.cuh"
 
@@ -192,24 +192,30 @@ __global__ void gate_mul_kernel(const T* __restrict__ a, const T* __restrict__ g
 
 // kind 1: the square of max(z, 0).  kPieces: 16 bytes a thread (width and ld multiples of a piece).
 template <typename T, bool kPieces>
-__global__ void unary_act_kernel(const T* __restrict__ z, long long ld, T* __restrict__ out, long long rows, int width,
-                                 int kind) {
+__global__ void unary_act_kernel(const T* __restrict__ z, long long ld, const float* __restrict__ bias, T* __restrict__ out,
+                                 long long rows, int width, int kind) {
   constexpr int V = kPieces ? 16 / static_cast<int>(sizeof(T)) : 1;
   wait_for_prior_kernels();
   launch_dependents();
   const long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * V;
   if (i >= rows * width) return;
-  const long long zi = (i / width) * ld + i % width;
+  const int c = static_cast<int>(i % width);
+  const long long zi = (i / width) * ld + c;
+  auto act = [&](float v, int j) {
+    if (bias != nullptr) v += bias[c + j];
+    if (kind == 2) return gelu_erf_f(v);
+    v = fmaxf(v, 0.0f);
+    return v * v;
+  };
   if (kPieces) {
     float v[V];
     load_piece<T, V>(v, z + zi);
 #pragma unroll
-    for (int j = 0; j < V; ++j) { v[j] = fmaxf(v[j], 0.0f); v[j] *= v[j]; }
+    for (int j = 0; j < V; ++j) v[j] = act(v[j], j);
     store_piece<T, V>(out + i, v);
     return;
   }
-  const float v = fmaxf(to_float<T>(z[zi]), 0.0f);
-  out[i] = from_float<T>(v * v);
+  out[i] = from_float<T>(act(to_float<T>(z[zi]), 0));
 }
 
 __global__ void scale_rows_kernel(float* __restrict__ x, long long n, float s) {
@@ -315,17 +321,18 @@ extern "C" int pih_gate_mul(int dtype, const void* a, const void* gate, long lon
 }
 
 // out [rows, width] contiguous = act(z [rows, ld]); kind 1: relu(z)^2
-extern "C" int pih_unary_act(int dtype, const void* z, long long ld, void* out, long long rows, int width, int kind,
-                             void* stream) {
+// bias: fp32 [width] or null, added first.  kind 1: the square of max(v, 0); 2: v / 2 (1 + erf(v / sqrt(2))).
+extern "C" int pih_unary_act(int dtype, const void* z, long long ld, const void* bias, void* out, long long rows, int width,
+                             int kind, void* stream) {
   if (rows <= 0 || width <= 0) return 0;
-  if (kind != 1) return PIH_ERR_BAD_ARGUMENT;
+  if (kind != 1 && kind != 2) return PIH_ERR_BAD_ARGUMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int V = dtype == PIH_F32 ? 4 : 8;
   const bool pieces = width % V == 0 && ld % V == 0 && aligned16(z) && aligned16(out);
   const long long n = rows * width / (pieces ? V : 1);
 #define PIH_UA(T, P)                                                                                                   \
   launch_kernel(unary_act_kernel<T, P>, flat_grid(n), dim3(256), 0, s, static_cast<const T*>(z), ld,                   \
-                static_cast<T*>(out), rows, width, kind)
+                static_cast<const float*>(bias), static_cast<T*>(out), rows, width, kind)
   if (dtype == PIH_BF16) { if (pieces) PIH_UA(bf16, true); else PIH_UA(bf16, false); }
   else if (dtype == PIH_F32) { if (pieces) PIH_UA(float, true); else PIH_UA(float, false); }
   else return PIH_ERR_BAD_ARGUMENT;

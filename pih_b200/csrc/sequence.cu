@@ -1,12 +1,14 @@
 // Kernels of mixers that carry a state from token to token, and of a residual stream kept in 32-bit.
 //
-//   embedding_stream      table rows (bf16 or fp32) -> a 32-bit stream
-//   rmsnorm_stream        h (fp32) += delta; out = h / sqrt(mean(h^2) + eps) * w, w a vector or ONE number
+//   embedding_stream      table rows (bf16 or fp32) times one number -> a 32-bit stream
+//   rmsnorm_stream        h (fp32) += scale * (delta + bias) (+ the token's embedding and a vector: a loop's next pass);
+//                         out = h / sqrt(mean(h^2) + eps) * w, w a vector or ONE number
 //   causal_conv           short causal convolution per channel over each request's rows, the last taps-1 inputs
 //                         carried in the request's state slot
-//   delta_prepare         unit-norm q and k per head, decay and write strength per head (32-bit)
+//   delta_prepare         unit-norm q and k per head, decay (one a head, or one a head and key channel) and write
+//                         strength per head (32-bit)
 //   delta_recurrence      gated delta rule: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
-//   gated_rmsnorm         per-head RMS norm of the read-out, times a weight, times silu(gate)
+//   gated_rmsnorm         per-head RMS norm of the read-out, times a weight, times silu(gate) or sigmoid(gate)
 //   rglru_gates, _chain   real-gated linear recurrent unit: S <- a S + sqrt(1 - a^2) (i u), out = S * gelu(y)
 //
 // A step's rows are packed: request r owns rows cu_q[r] .. cu_q[r+1]-1 in the order of their positions, and
@@ -21,15 +23,13 @@ namespace pih {
 
 constexpr int kMaxTaps = 16;
 
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
 template <typename T>
 __global__ void embedding_stream_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out,
-                                        int hidden, int vocab, uint32_t* err) {
+                                        int hidden, int vocab, float scale, uint32_t* err) {
   wait_for_prior_kernels();
   launch_dependents();
   const int row = blockIdx.x;
@@ -40,37 +40,161 @@ __global__ void embedding_stream_kernel(const T* __restrict__ table, const int* 
     id = 0;
   }
   for (int c = threadIdx.x; c < hidden; c += blockDim.x)
-    out[static_cast<long long>(row) * hidden + c] = bad ? 0.0f : to_float<T>(table[static_cast<long long>(id) * hidden + c]);
+    out[static_cast<long long>(row) * hidden + c] = bad ? 0.0f : to_float<T>(table[static_cast<long long>(id) * hidden + c]) * scale;
 }
 
-// One block a row.  Without ``rows``: h[row] += delta[row] is stored back and normed.  With ``rows`` (a gather of the
-// rows whose logits are wanted) nothing is stored: the sum is formed for the norm alone.
-template <typename TD, typename TO>
-__global__ void __launch_bounds__(256)
-rmsnorm_stream_kernel(float* __restrict__ h, const TD* __restrict__ delta, const float* __restrict__ weight, int weight_len,
+// What is added to a row of the stream before it is normed: scale * (delta + bias), then, where a loop's next pass
+// begins, table_scale * table[ids[row]] (the token's embedding once more) and a vector.  Null pointers: absent.
+template <typename TD>
+struct StreamAdd {
+  const TD* delta;
+  float scale;
+  const float* bias;
+  const TD* table;
+  const int* ids;
+  int vocab;
+  float table_scale;
+  const float* vec;
+};
+
+// ``n`` (V) neighbouring columns as one 16-byte load where V is 4
+template <int V>
+__device__ __forceinline__ void load_floats(float (&v)[V], const float* src) {
+  if constexpr (V == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(src);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = src[i];
+  }
+}
+template <int V>
+__device__ __forceinline__ void load_floats(float (&v)[V], const __nv_bfloat16* src) {
+  if constexpr (V == 4) {
+    const uint2 w = *reinterpret_cast<const uint2*>(src);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = __bfloat162float(src[i]);
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_floats(float* dst, const float (&v)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+  else
+#pragma unroll
+    for (int i = 0; i < V; ++i) dst[i] = v[i];
+}
+template <int V>
+__device__ __forceinline__ void store_floats(__nv_bfloat16* dst, const float (&v)[V]) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) dst[i] = __float2bfloat16_rn(v[i]);
+  }
+}
+
+// The new values of columns c .. c + V - 1 of a row (32-bit sums).
+template <typename TD, int V>
+__device__ __forceinline__ void stream_sum(float (&v)[V], const float* hr, const TD* dr, const TD* er, const StreamAdd<TD>& add,
+                                           int c) {
+  load_floats<V>(v, hr + c);
+  if (dr != nullptr) {
+    float d[V];
+    load_floats<V>(d, dr + c);
+    if (add.bias != nullptr) {
+      float b[V];
+      load_floats<V>(b, add.bias + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) d[i] += b[i];
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = fmaf(add.scale, d[i], v[i]);
+  }
+  if (er != nullptr) {
+    float e[V];
+    load_floats<V>(e, er + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = fmaf(add.table_scale, e[i], v[i]);
+  }
+  if (add.vec != nullptr) {
+    float e[V];
+    load_floats<V>(e, add.vec + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] += e[i];
+  }
+}
+
+// One block a row.  Without ``rows`` the row's new sum is stored back and normed; with ``rows`` (a gather of the rows whose
+// logits are wanted) nothing is stored: the sum is formed for the norm alone.  V columns a thread at a time; the first
+// kHeld pieces of a thread stay in registers between the sum of squares and the writing, later ones are formed (or read)
+// again.
+template <typename TD, typename TO, int V>
+__global__ void __launch_bounds__(512)
+rmsnorm_stream_kernel(float* __restrict__ h, const StreamAdd<TD> add, const float* __restrict__ weight, int weight_len,
                       TO* __restrict__ out, const int* __restrict__ rows, int width, float eps) {
+  constexpr int kHeld = 4;
   __shared__ float scratch[33];
   wait_for_prior_kernels();
   launch_dependents();
   const int row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
   float* hr = h + static_cast<long long>(row) * width;
-  const TD* dr = delta != nullptr ? delta + static_cast<long long>(row) * width : nullptr;
+  const TD* dr = add.delta != nullptr ? add.delta + static_cast<long long>(row) * width : nullptr;
+  const TD* er = nullptr;
+  if (add.table != nullptr) {
+    const int id = add.ids[row];                               // (a bad id was reported by the embedding)
+    er = add.table + static_cast<long long>(id >= 0 && id < add.vocab ? id : 0) * width;
+  }
+  const bool changes = dr != nullptr || er != nullptr || add.vec != nullptr;
+  const int step = static_cast<int>(blockDim.x) * V, c0 = static_cast<int>(threadIdx.x) * V;
+  float held[kHeld][V];
   float ss = 0.0f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    float v = hr[c];
-    if (dr != nullptr) {
-      v += to_float<TD>(dr[c]);
-      if (rows == nullptr) hr[c] = v;
+#pragma unroll
+  for (int u = 0; u < kHeld; ++u) {
+    const int c = c0 + u * step;
+    if (c < width) {
+      stream_sum<TD, V>(held[u], hr, dr, er, add, c);
+      if (changes && rows == nullptr) store_floats<V>(hr + c, held[u]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(held[u][i], held[u][i], ss);
     }
-    ss = fmaf(v, v, ss);
+  }
+  for (int c = c0 + kHeld * step; c < width; c += step) {
+    float v[V];
+    stream_sum<TD, V>(v, hr, dr, er, add, c);
+    if (changes && rows == nullptr) store_floats<V>(hr + c, v);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
   }
   ss = block_sum(ss, scratch);
   const float scale = 1.0f / sqrtf(ss / static_cast<float>(width) + eps);
   TO* o = out + static_cast<long long>(blockIdx.x) * width;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    float v = hr[c];
-    if (dr != nullptr && rows != nullptr) v += to_float<TD>(dr[c]);
-    o[c] = from_float<TO>(v * scale * (weight_len == 1 ? weight[0] : weight[c]));
+  auto write = [&](float (&v)[V], int c) {
+    float w[V];
+    if (weight_len == 1) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) w[i] = weight[0];
+    } else {
+      load_floats<V>(w, weight + c);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = v[i] * scale * w[i];
+    store_floats<V>(o + c, v);
+  };
+#pragma unroll
+  for (int u = 0; u < kHeld; ++u) {
+    const int c = c0 + u * step;
+    if (c < width) write(held[u], c);
+  }
+  for (int c = c0 + kHeld * step; c < width; c += step) {
+    float v[V];
+    if (rows == nullptr) load_floats<V>(v, hr + c);            // (the thread's own store)
+    else stream_sum<TD, V>(v, hr, dr, er, add, c);
+    write(v, c);
   }
 }
 
@@ -164,11 +288,13 @@ causal_conv_history_kernel(const T* __restrict__ x, long long ldx, const float* 
 }
 
 // One block a row.  qk: [rows, ld] with q heads at column 0 and k heads at column kv_heads*dim (after convolution and
-// activation); ba: [rows, ldb] with the write-strength logits at column 0 and the decay logits at column ``heads``.
-// qn, kn: fp32 [rows, kv_heads, dim]; decay (as g - 1), beta: fp32 [rows, heads].
-template <typename T>
+// activation); b: [rows, ldb] write-strength logits a head; a: [rows, lda] decay logits, one a head or (``channels``) one a
+// head and key channel, [heads, dim], with a bias of the same layout; decay_log: one a head.
+// qn, kn: fp32 [rows, kv_heads, dim]; decay (as g - 1): fp32 [rows, heads] or [rows, heads, dim]; beta: fp32 [rows, heads].
+template <typename T, typename TA>
 __global__ void __launch_bounds__(128)
-delta_prepare_kernel(const T* __restrict__ qk, long long ld, const T* __restrict__ ba, long long ldb,
+delta_prepare_kernel(const T* __restrict__ qk, long long ld, const T* __restrict__ b, long long ldb,
+                     const TA* __restrict__ a, long long lda, int channels,
                      const float* __restrict__ decay_log, const float* __restrict__ decay_bias, float* __restrict__ qn,
                      float* __restrict__ kn, float* __restrict__ decay, float* __restrict__ beta, int heads, int kv_heads,
                      int dim, float unit_eps, float q_scale) {
@@ -186,17 +312,19 @@ delta_prepare_kernel(const T* __restrict__ qk, long long ld, const T* __restrict
     for (int i = lane; i < dim; i += 32) dst[i] = to_float<T>(src[i]) * scale;
   }
   for (int h = threadIdx.x; h < heads; h += blockDim.x) {
-    const float b = to_float<T>(ba[static_cast<long long>(row) * ldb + h]);
-    const float a = to_float<T>(ba[static_cast<long long>(row) * ldb + heads + h]);
-    beta[static_cast<long long>(row) * heads + h] = sigmoid_f(b);
-    // g - 1 rather than g: a decay next to 1 keeps its distance from 1 to full precision (see rglru_scan_kernel)
-    decay[static_cast<long long>(row) * heads + h] = expm1f(-expf(decay_log[h]) * softplus_f(a + decay_bias[h]));
+    beta[static_cast<long long>(row) * heads + h] = sigmoid_f(to_float<T>(b[static_cast<long long>(row) * ldb + h]));
   }
+  // g - 1 rather than g: a decay next to 1 keeps its distance from 1 to full precision (see rglru_gates_kernel)
+  const int per = channels ? dim : 1;
+  const long long row_a = static_cast<long long>(row) * lda, row_g = static_cast<long long>(row) * heads * per;
+  for (int i = threadIdx.x; i < heads * per; i += blockDim.x)
+    decay[row_g + i] = expm1f(-expf(decay_log[i / per]) * softplus_f(to_float<TA>(a[row_a + i]) + decay_bias[i]));
 }
 
 // Block (request, head, slice of value columns); thread j owns column v0 + j of S (all ``dim`` rows, in shared memory:
-// S[i][j], conflict-free).  The next token's k and q are fetched into registers while this token is computed.
-template <typename T>
+// S[i][j], conflict-free).  The next token's k and q (and, with kChannel, its decay a key channel) are fetched into
+// registers while this token is computed.
+template <typename T, bool kChannel>
 __global__ void delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const T* __restrict__ v,
                                         long long ldv, const float* __restrict__ decay, const float* __restrict__ beta,
                                         float* __restrict__ out, float* __restrict__ state, long long state_stride,
@@ -213,59 +341,68 @@ __global__ void delta_recurrence_kernel(const float* __restrict__ qn, const floa
   if (hi <= lo || slot < 0) return;
   const int kh = h / (heads / kv_heads);
   float* S = smem;                          // [dim][cols]
-  float* kq = smem + dim * cols;            // [2 buffers][k: dim | q: dim]
+  constexpr int kVecs = kChannel ? 3 : 2;
+  float* kq = smem + dim * cols;            // [2 buffers][k: dim | q: dim | decay - 1: dim]
   const bool live = col < vdim;
   float* Sg = state + slot * state_stride + (static_cast<long long>(h) * dim) * vdim;
   for (int i = 0; i < dim; ++i) S[i * cols + j] = live ? Sg[static_cast<long long>(i) * vdim + col] : 0.0f;
-  const int per = (2 * dim + cols - 1) / cols;                   // numbers of k|q a thread fetches
+  const int per = (kVecs * dim + cols - 1) / cols;               // numbers of k|q|decay a thread fetches
   auto fetch = [&](int t, int e) -> float {
     const int idx = j + e * cols;
-    if (idx >= 2 * dim) return 0.0f;
+    if (idx >= kVecs * dim) return 0.0f;
+    if (kChannel && idx >= 2 * dim) return decay[(static_cast<long long>(t) * heads + h) * dim + (idx - 2 * dim)];
     const float* src = idx < dim ? kn : qn;
     return src[(static_cast<long long>(t) * kv_heads + kh) * dim + (idx < dim ? idx : idx - dim)];
   };
-  constexpr int kMaxPer = 16;               // dim <= 8 * cols
+  constexpr int kMaxPer = 8 * kVecs;        // dim <= 8 * cols
   float nxt[kMaxPer];
 #pragma unroll
   for (int e = 0; e < kMaxPer; ++e) nxt[e] = e < per ? fetch(lo, e) : 0.0f;
   for (int t = lo; t < hi; ++t) {
-    float* cur = kq + (t & 1) * 2 * dim;
+    float* cur = kq + (t & 1) * kVecs * dim;
 #pragma unroll
     for (int e = 0; e < kMaxPer; ++e)
-      if (e < per && j + e * cols < 2 * dim) cur[j + e * cols] = nxt[e];
+      if (e < per && j + e * cols < kVecs * dim) cur[j + e * cols] = nxt[e];
     __syncthreads();
     if (t + 1 < hi) {
 #pragma unroll
       for (int e = 0; e < kMaxPer; ++e) nxt[e] = e < per ? fetch(t + 1, e) : 0.0f;
     }
-    const float gm1 = decay[static_cast<long long>(t) * heads + h];        // g - 1; g x is formed as x + (g - 1) x
     const float b = beta[static_cast<long long>(t) * heads + h];
     const float vj = live ? to_float<T>(v[static_cast<long long>(t) * ldv + static_cast<long long>(h) * vdim + col]) : 0.0f;
     const float* k = cur;
     const float* q = cur + dim;
+    // g - 1; g x is formed as x + (g - 1) x.  One decay a head multiplies the finished dot product, one a key channel the
+    // rows of S first
+    const float* gc = cur + 2 * dim;
+    const float gm1 = kChannel ? 0.0f : decay[static_cast<long long>(t) * heads + h];
+    auto decayed = [&](int i) {
+      const float x = S[i * cols + j];
+      return fmaf(kChannel ? gc[i] : gm1, x, x);
+    };
     float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
     int i = 0;
     for (; i + 4 <= dim; i += 4) {
-      a0 = fmaf(S[(i + 0) * cols + j], k[i + 0], a0);
-      a1 = fmaf(S[(i + 1) * cols + j], k[i + 1], a1);
-      a2 = fmaf(S[(i + 2) * cols + j], k[i + 2], a2);
-      a3 = fmaf(S[(i + 3) * cols + j], k[i + 3], a3);
+      a0 = fmaf(kChannel ? decayed(i + 0) : S[(i + 0) * cols + j], k[i + 0], a0);
+      a1 = fmaf(kChannel ? decayed(i + 1) : S[(i + 1) * cols + j], k[i + 1], a1);
+      a2 = fmaf(kChannel ? decayed(i + 2) : S[(i + 2) * cols + j], k[i + 2], a2);
+      a3 = fmaf(kChannel ? decayed(i + 3) : S[(i + 3) * cols + j], k[i + 3], a3);
     }
-    for (; i < dim; ++i) a0 = fmaf(S[i * cols + j], k[i], a0);
+    for (; i < dim; ++i) a0 = fmaf(kChannel ? decayed(i) : S[i * cols + j], k[i], a0);
     const float dot = (a0 + a1) + (a2 + a3);
-    const float u = b * (vj - fmaf(gm1, dot, dot));
+    const float u = b * (vj - (kChannel ? dot : fmaf(gm1, dot, dot)));
     float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
     i = 0;
     for (; i + 4 <= dim; i += 4) {
-      const float s0 = fmaf(k[i + 0], u, fmaf(gm1, S[(i + 0) * cols + j], S[(i + 0) * cols + j]));
-      const float s1 = fmaf(k[i + 1], u, fmaf(gm1, S[(i + 1) * cols + j], S[(i + 1) * cols + j]));
-      const float s2 = fmaf(k[i + 2], u, fmaf(gm1, S[(i + 2) * cols + j], S[(i + 2) * cols + j]));
-      const float s3 = fmaf(k[i + 3], u, fmaf(gm1, S[(i + 3) * cols + j], S[(i + 3) * cols + j]));
+      const float s0 = fmaf(k[i + 0], u, decayed(i + 0));
+      const float s1 = fmaf(k[i + 1], u, decayed(i + 1));
+      const float s2 = fmaf(k[i + 2], u, decayed(i + 2));
+      const float s3 = fmaf(k[i + 3], u, decayed(i + 3));
       S[(i + 0) * cols + j] = s0; S[(i + 1) * cols + j] = s1; S[(i + 2) * cols + j] = s2; S[(i + 3) * cols + j] = s3;
       o0 = fmaf(s0, q[i + 0], o0); o1 = fmaf(s1, q[i + 1], o1); o2 = fmaf(s2, q[i + 2], o2); o3 = fmaf(s3, q[i + 3], o3);
     }
     for (; i < dim; ++i) {
-      const float s0 = fmaf(k[i], u, fmaf(gm1, S[i * cols + j], S[i * cols + j]));
+      const float s0 = fmaf(k[i], u, decayed(i));
       S[i * cols + j] = s0;
       o0 = fmaf(s0, q[i], o0);
     }
@@ -291,22 +428,32 @@ __device__ __forceinline__ void async_copy_4(void* smem_dst, const void* src) {
 __device__ __forceinline__ void async_copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void async_copies_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-template <typename T, int kDim>
-__global__ void __launch_bounds__(kDim >= 64 ? 256 : 128)
+// With kChannel the decay (as g - 1, [rows, heads, kDim]) multiplies the rows of S; it is staged like k and q.
+template <int kDim, bool kChannel>
+struct DeltaShape {
+  static constexpr int kParts = kDim >= 256 && kChannel ? 16 : (kDim >= 64 ? 8 : 4);   // threads a column of S
+  static constexpr int kThreads = 32 * kParts;
+  static constexpr int kRows = kDim / kParts;             // rows of S a thread holds
+  static constexpr int kSeg = kRows + 4;                  // a part's stretch of k (or q) in the staging buffer: the parts'
+                                                          // 16-byte reads fall into different banks
+  static constexpr int kVecs = kChannel ? 3 : 2;          // vectors of kDim numbers staged a token: k | q (| decay - 1)
+  static constexpr int kChunk = kDim <= 128 ? 16 : 8;     // tokens staged at a time (even)
+};
+
+template <typename T, int kDim, bool kChannel>
+__global__ void __launch_bounds__(DeltaShape<kDim, kChannel>::kThreads)
 delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const T* __restrict__ v,
                             long long ldv, const float* __restrict__ decay, const float* __restrict__ beta,
                             float* __restrict__ out, float* __restrict__ state, long long state_stride,
                             const int* __restrict__ cu_q, const int* __restrict__ state_slots, int heads, int kv_heads,
                             int vdim) {
-  constexpr int kParts = kDim >= 64 ? 8 : 4;              // threads a column of S
-  constexpr int kThreads = 32 * kParts;
-  constexpr int kRows = kDim / kParts;                    // rows of S a thread holds
-  constexpr int kSeg = kRows + 4;                         // a part's stretch of k (or q) in the staging buffer: the parts'
-                                                          // 16-byte reads fall into different banks
-  constexpr int kChunk = kDim <= 128 ? 16 : 8;            // tokens staged at a time (even)
+  typedef DeltaShape<kDim, kChannel> Shape;
+  constexpr int kParts = Shape::kParts, kThreads = Shape::kThreads, kRows = Shape::kRows, kSeg = Shape::kSeg;
+  constexpr int kVecs = Shape::kVecs, kChunk = Shape::kChunk;
   constexpr int kVWords = 32 * sizeof(T) / 4;             // the block's 32 values of a token, in 32-bit words
-  constexpr int kTok = 2 * kParts * kSeg + 4 + kVWords;   // words staged a token: k | q | decay - 1, write strength, pad | values
-  constexpr int kCopies = 2 * (kDim / 4) + 2 + kVWords;   // asynchronous copies a token
+  constexpr int kTail = kVecs * kParts * kSeg;            // where what is not a vector of kDim numbers begins
+  constexpr int kTok = kTail + 4 + kVWords;               // words staged a token: vectors | decay - 1, write strength, pad | values
+  constexpr int kCopies = kVecs * (kDim / 4) + 2 + kVWords;   // asynchronous copies a token
   extern __shared__ __align__(16) float stage[];          // [2][kChunk][kTok]
   wait_for_prior_kernels();
   launch_dependents();
@@ -329,26 +476,28 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
       const int tok = i / kCopies, c = i - tok * kCopies;
       const int t = t0 + tok;
       float* dst = stage + (b * kChunk + tok) * kTok;
-      if (c < 2 * (kDim / 4)) {
-        const bool is_q = c >= kDim / 4;
-        const int e = (is_q ? c - kDim / 4 : c) * 4;             // element of k (or q)
-        const float* src = (is_q ? qn : kn) + (static_cast<long long>(t) * kv_heads + kh) * kDim + e;
-        async_copy_16(dst + (is_q ? kParts * kSeg : 0) + (e / kRows) * kSeg + e % kRows, src);
-      } else if (c < 2 * (kDim / 4) + 2) {
-        const int which = c - 2 * (kDim / 4);
-        async_copy_4(dst + 2 * kParts * kSeg + which, (which ? beta : decay) + static_cast<long long>(t) * heads + h);
+      if (c < kVecs * (kDim / 4)) {
+        const int which = c / (kDim / 4);                        // 0: k, 1: q, 2: the decay a channel
+        const int e = (c - which * (kDim / 4)) * 4;              // element of it
+        const float* src = which == 2 ? decay + (static_cast<long long>(t) * heads + h) * kDim + e
+                                      : (which == 1 ? qn : kn) + (static_cast<long long>(t) * kv_heads + kh) * kDim + e;
+        async_copy_16(dst + which * kParts * kSeg + (e / kRows) * kSeg + e % kRows, src);
+      } else if (c < kVecs * (kDim / 4) + 2) {
+        const int which = c - kVecs * (kDim / 4);
+        if (which == 1 || !kChannel)
+          async_copy_4(dst + kTail + which, (which ? beta : decay) + static_cast<long long>(t) * heads + h);
       } else {
-        const int w = c - 2 * (kDim / 4) - 2;                    // word w holds 4 / sizeof(T) values
+        const int w = c - kVecs * (kDim / 4) - 2;                // word w holds 4 / sizeof(T) values
         const int first_col = col0 + w * (4 / static_cast<int>(sizeof(T)));
         if (first_col < vdim)
-          async_copy_4(dst + 2 * kParts * kSeg + 4 + w,
+          async_copy_4(dst + kTail + 4 + w,
                        v + static_cast<long long>(t) * ldv + static_cast<long long>(h) * vdim + first_col);
       }
     }
     async_copies_commit();
   };
   // a token's numbers from the staging buffer into registers, one token ahead of the arithmetic
-  struct Tok { float k[kRows], q[kRows], gm1, b, v; };
+  struct Tok { float k[kRows], q[kRows], g[kChannel ? kRows : 1], b, v; };
   auto load = [&](Tok& x, const float* cur) {
 #pragma unroll
     for (int i = 0; i < kRows; i += 4) {
@@ -356,18 +505,27 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
       const float4 q4 = *reinterpret_cast<const float4*>(cur + kParts * kSeg + part * kSeg + i);
       x.k[i] = k4.x; x.k[i + 1] = k4.y; x.k[i + 2] = k4.z; x.k[i + 3] = k4.w;
       x.q[i] = q4.x; x.q[i + 1] = q4.y; x.q[i + 2] = q4.z; x.q[i + 3] = q4.w;
+      if constexpr (kChannel) {
+        const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kParts * kSeg + part * kSeg + i);
+        x.g[i] = g4.x; x.g[i + 1] = g4.y; x.g[i + 2] = g4.z; x.g[i + 3] = g4.w;
+      }
     }
-    x.gm1 = cur[2 * kParts * kSeg];
-    x.b = cur[2 * kParts * kSeg + 1];
-    x.v = to_float<T>(reinterpret_cast<const T*>(cur + 2 * kParts * kSeg + 4)[cl]);
+    if constexpr (!kChannel) x.g[0] = cur[kTail];
+    x.b = cur[kTail + 1];
+    x.v = to_float<T>(reinterpret_cast<const T*>(cur + kTail + 4)[cl]);
   };
   auto reduce = [&](float x) {
     x += __shfl_xor_sync(0xffffffffu, x, 1);
     x += __shfl_xor_sync(0xffffffffu, x, 2);
-    if (kParts == 8) x += __shfl_xor_sync(0xffffffffu, x, 4);
+    if (kParts >= 8) x += __shfl_xor_sync(0xffffffffu, x, 4);
+    if (kParts >= 16) x += __shfl_xor_sync(0xffffffffu, x, 8);
     return x;
   };
   auto compute = [&](const Tok& x, int t) {
+    if constexpr (kChannel) {
+#pragma unroll
+      for (int i = 0; i < kRows; ++i) S[i] = fmaf(x.g[i], S[i], S[i]);
+    }
     float a0 = 0.0f, a1 = 0.0f;
 #pragma unroll
     for (int i = 0; i < kRows; i += 2) {
@@ -375,12 +533,12 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
       a1 = fmaf(S[i + 1], x.k[i + 1], a1);
     }
     const float dot = reduce(a0 + a1);
-    const float u = x.b * (x.v - fmaf(x.gm1, dot, dot));
+    const float u = x.b * (x.v - (kChannel ? dot : fmaf(x.g[0], dot, dot)));
     float o0 = 0.0f, o1 = 0.0f;
 #pragma unroll
     for (int i = 0; i < kRows; i += 2) {
-      S[i] = fmaf(x.k[i], u, fmaf(x.gm1, S[i], S[i]));
-      S[i + 1] = fmaf(x.k[i + 1], u, fmaf(x.gm1, S[i + 1], S[i + 1]));
+      S[i] = fmaf(x.k[i], u, kChannel ? S[i] : fmaf(x.g[0], S[i], S[i]));
+      S[i + 1] = fmaf(x.k[i + 1], u, kChannel ? S[i + 1] : fmaf(x.g[0], S[i + 1], S[i + 1]));
       o0 = fmaf(S[i], x.q[i], o0);
       o1 = fmaf(S[i + 1], x.q[i + 1], o1);
     }
@@ -415,11 +573,13 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
   }
 }
 
-// One warp a (row, head): o fp32 [rows, heads, vdim]; gate [rows, ldg] with head h at column h * vdim.
-template <typename T>
+// One warp a (row, head): o fp32 [rows, heads, vdim]; gate [rows, ldg] and out [rows, ldo] with head h at column h * vdim.
+// activation 0: silu(gate), 1: sigmoid(gate); out_scale multiplies.
+template <typename TG, typename T>
 __global__ void __launch_bounds__(128)
-gated_rmsnorm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ldg, const float* __restrict__ weight,
-                     T* __restrict__ out, long long rows_heads, int heads, int vdim, float eps) {
+gated_rmsnorm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, long long ldg, const float* __restrict__ weight,
+                     T* __restrict__ out, long long ldo, long long rows_heads, int heads, int vdim, float eps, int activation,
+                     float out_scale) {
   wait_for_prior_kernels();
   launch_dependents();
   const long long item = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -431,12 +591,12 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const T* __restrict__ gate, lo
   float ss = 0.0f;
   for (int i = lane; i < vdim; i += 32) ss = fmaf(src[i], src[i], ss);
   ss = warp_sum(ss);
-  const float scale = 1.0f / sqrtf(ss / static_cast<float>(vdim) + eps);
-  const T* g = gate + row * ldg + static_cast<long long>(h) * vdim;
-  T* dst = out + item * vdim;
+  const float scale = 1.0f / sqrtf(ss / static_cast<float>(vdim) + eps) * out_scale;
+  const TG* g = gate + row * ldg + static_cast<long long>(h) * vdim;
+  T* dst = out + row * ldo + static_cast<long long>(h) * vdim;
   for (int i = lane; i < vdim; i += 32) {
-    const float z = to_float<T>(g[i]);
-    dst[i] = from_float<T>(src[i] * scale * weight[i] * (z / (1.0f + expf(-z))));
+    const float z = to_float<TG>(g[i]);
+    dst[i] = from_float<T>(src[i] * scale * weight[i] * ((activation == 1 ? 1.0f : z) / (1.0f + expf(-z))));
   }
 }
 
@@ -516,39 +676,61 @@ using namespace pih;
 typedef __nv_bfloat16 bf16;
 
 extern "C" int pih_embedding_stream(int dtype, const void* table, const void* ids, void* out, int rows, int hidden,
-                                    int vocab, void* err, void* stream) {
+                                    int vocab, float scale, void* err, void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int threads = hidden >= 256 ? 256 : 64;
   if (dtype == PIH_F32)
     launch_kernel(embedding_stream_kernel<float>, dim3(rows), dim3(threads), 0, s, static_cast<const float*>(table),
-                  static_cast<const int*>(ids), static_cast<float*>(out), hidden, vocab, static_cast<uint32_t*>(err));
+                  static_cast<const int*>(ids), static_cast<float*>(out), hidden, vocab, scale, static_cast<uint32_t*>(err));
   else if (dtype == PIH_BF16)
     launch_kernel(embedding_stream_kernel<bf16>, dim3(rows), dim3(threads), 0, s, static_cast<const bf16*>(table),
-                  static_cast<const int*>(ids), static_cast<float*>(out), hidden, vocab, static_cast<uint32_t*>(err));
+                  static_cast<const int*>(ids), static_cast<float*>(out), hidden, vocab, scale, static_cast<uint32_t*>(err));
   else
     return PIH_ERR_BAD_ARGUMENT;
   PIH_LAUNCH_CHECK();
   return 0;
 }
 
-extern "C" int pih_rmsnorm_stream(int delta_dtype, int out_dtype, void* h, const void* delta, const void* weight,
-                                  int weight_len, void* out, const void* rows, int n_out, int width, float eps,
-                                  void* stream) {
+// h [.., width] fp32: h += delta_scale * (delta + bias), then += table_scale * table[ids[row]] (where table is given: of
+// the delta's dtype, [vocab, width]) and += vec (fp32 [width]); out: the normed rows.  delta, bias, table, vec nullable; a
+// bias comes with a delta only.
+extern "C" int pih_rmsnorm_stream(int delta_dtype, int out_dtype, void* h, const void* delta, float delta_scale,
+                                  const void* bias, const void* table, const void* ids, int vocab, float table_scale,
+                                  const void* vec, const void* weight, int weight_len, void* out, const void* rows, int n_out,
+                                  int width, float eps, void* stream) {
   if (n_out <= 0) return 0;
   if (weight_len != 1 && weight_len != width) return PIH_ERR_BAD_ARGUMENT;
+  if ((bias != nullptr && delta == nullptr) || (table != nullptr && (ids == nullptr || vocab < 1))) return PIH_ERR_BAD_ARGUMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int threads = width >= 1024 ? 256 : 128;
+  auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool four = width % 4 == 0 && aligned(h) && aligned(delta) && aligned(bias) && aligned(table) && aligned(vec) &&
+                    aligned(weight) && aligned(out);
+  const int threads = width <= 512 ? 128 : (width <= 4096 ? 256 : 512);
+#define PIH_NORM_V(TD, TO, V)                                                                                         \
+  do {                                                                                                                \
+    StreamAdd<TD> add;                                                                                                \
+    add.delta = static_cast<const TD*>(delta);                                                                        \
+    add.scale = delta_scale;                                                                                          \
+    add.bias = static_cast<const float*>(bias);                                                                       \
+    add.table = static_cast<const TD*>(table);                                                                        \
+    add.ids = static_cast<const int*>(ids);                                                                           \
+    add.vocab = vocab;                                                                                                \
+    add.table_scale = table_scale;                                                                                    \
+    add.vec = static_cast<const float*>(vec);                                                                         \
+    launch_kernel(rmsnorm_stream_kernel<TD, TO, V>, dim3(n_out), dim3(threads), 0, s, static_cast<float*>(h), add,     \
+                  static_cast<const float*>(weight), weight_len, static_cast<TO*>(out), static_cast<const int*>(rows), \
+                  width, eps);                                                                                        \
+  } while (0)
 #define PIH_NORM(TD, TO)                                                                                              \
-  launch_kernel(rmsnorm_stream_kernel<TD, TO>, dim3(n_out), dim3(threads), 0, s, static_cast<float*>(h),               \
-                static_cast<const TD*>(delta), static_cast<const float*>(weight), weight_len, static_cast<TO*>(out),   \
-                static_cast<const int*>(rows), width, eps)
+  do { if (four) PIH_NORM_V(TD, TO, 4); else PIH_NORM_V(TD, TO, 1); } while (0)
   if (delta_dtype == PIH_F32 && out_dtype == PIH_F32) PIH_NORM(float, float);
   else if (delta_dtype == PIH_BF16 && out_dtype == PIH_BF16) PIH_NORM(bf16, bf16);
   else if (delta_dtype == PIH_F32 && out_dtype == PIH_BF16) PIH_NORM(float, bf16);
   else if (delta_dtype == PIH_BF16 && out_dtype == PIH_F32) PIH_NORM(bf16, float);
   else return PIH_ERR_BAD_ARGUMENT;
 #undef PIH_NORM
+#undef PIH_NORM_V
   PIH_LAUNCH_CHECK();
   return 0;
 }
@@ -584,85 +766,111 @@ extern "C" int pih_causal_conv(int dtype, const void* x, long long ldx, const vo
 }
 
 // The gated delta rule over a step's rows.  qkv [rows, ld]: q heads, k heads, v heads (after convolution and SiLU);
-// ba [rows, ldb]: write-strength logits, decay logits.  scratch: fp32, rows * (2 * kv_heads * dim + 2 * heads).
-// out: fp32 [rows, heads, vdim].  The state S [heads, dim, vdim] lies at the start of a request's slot.
-extern "C" int pih_gated_delta_rule(int dtype, const void* qkv, long long ld, const void* ba, long long ldb,
-                                    const void* decay_log, const void* decay_bias, void* scratch, void* out, void* state,
-                                    long long state_stride, const void* cu_q, const void* state_slots, int rows,
-                                    int requests, int heads, int kv_heads, int dim, int vdim, float unit_eps,
-                                    float q_scale, void* stream) {
-  if (rows <= 0 || requests <= 0) return 0;
-  if (heads % kv_heads) return PIH_ERR_BAD_ARGUMENT;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int cols = vdim >= 64 ? 64 : 32;
-  if (dim > 8 * cols) return PIH_ERR_UNSUPPORTED;
-  const size_t smem = (static_cast<size_t>(dim) * cols + 4 * static_cast<size_t>(dim)) * sizeof(float);
-  if (smem > 200 * 1024) return PIH_ERR_UNSUPPORTED;
-  float* qn = static_cast<float*>(scratch);
-  float* kn = qn + static_cast<long long>(rows) * kv_heads * dim;
-  float* decay = kn + static_cast<long long>(rows) * kv_heads * dim;
-  float* beta = decay + static_cast<long long>(rows) * heads;
-  dim3 grid(requests, heads, (vdim + cols - 1) / cols);
-  if (grid.y > 65535 || grid.z > 65535) return PIH_ERR_UNSUPPORTED;
-  const long long qk_size = static_cast<long long>(kv_heads) * dim;
-  int dim_instance = dim;
-#define PIH_DELTA_REG(T, D)                                                                                            \
-  do {                                                                                                                 \
-    const int parts = (D) >= 64 ? 8 : 4;                                                                               \
-    const size_t staged = 2 * static_cast<size_t>((D) <= 128 ? 16 : 8) *                                               \
-                          (2 * parts * ((D) / parts + 4) + 4 + 32 * sizeof(T) / 4) * sizeof(float);                    \
-    if (staged > 48 * 1024)                                                                                            \
-      cudaFuncSetAttribute(delta_recurrence_reg_kernel<T, D>, cudaFuncAttributeMaxDynamicSharedMemorySize,             \
-                           static_cast<int>(staged));                                                                  \
-    launch_kernel(delta_recurrence_reg_kernel<T, D>, dim3(requests, heads, (vdim + 31) / 32), dim3(32 * parts), staged, s, \
-                  static_cast<const float*>(qn), static_cast<const float*>(kn),                                        \
-                  static_cast<const T*>(qkv) + 2 * qk_size, ld, static_cast<const float*>(decay),                      \
-                  static_cast<const float*>(beta), static_cast<float*>(out), static_cast<float*>(state), state_stride, \
-                  static_cast<const int*>(cu_q), static_cast<const int*>(state_slots), heads, kv_heads, vdim);         \
-  } while (0)
-#define PIH_DELTA(T)                                                                                                   \
-  do {                                                                                                                 \
-    launch_kernel(delta_prepare_kernel<T>, dim3(rows), dim3(128), 0, s, static_cast<const T*>(qkv), ld,                \
-                  static_cast<const T*>(ba), ldb, static_cast<const float*>(decay_log),                                \
-                  static_cast<const float*>(decay_bias), qn, kn, decay, beta, heads, kv_heads, dim, unit_eps, q_scale); \
-    PIH_LAUNCH_CHECK();                                                                                                \
-    const bool words = sizeof(T) == 4 || (ld % 2 == 0 && vdim % 2 == 0);      /* values are copied in 32-bit words */  \
-    if (!words) dim_instance = 0;                                                                                      \
-    if (dim_instance == 16) PIH_DELTA_REG(T, 16);                                                                      \
-    else if (dim_instance == 32) PIH_DELTA_REG(T, 32);                                                                          \
-    else if (dim_instance == 64) PIH_DELTA_REG(T, 64);                                                                          \
-    else if (dim_instance == 128) PIH_DELTA_REG(T, 128);                                                                        \
-    else if (dim_instance == 256) PIH_DELTA_REG(T, 256);                                                                        \
-    else {                                                                                                             \
-      if (smem > 48 * 1024)                                                                                            \
-        cudaFuncSetAttribute(delta_recurrence_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)); \
-      launch_kernel(delta_recurrence_kernel<T>, grid, dim3(cols), smem, s, static_cast<const float*>(qn),              \
-                    static_cast<const float*>(kn), static_cast<const T*>(qkv) + 2 * qk_size, ld,                       \
-                    static_cast<const float*>(decay), static_cast<const float*>(beta), static_cast<float*>(out),       \
-                    static_cast<float*>(state), state_stride, static_cast<const int*>(cu_q),                           \
-                    static_cast<const int*>(state_slots), heads, kv_heads, dim, vdim);                                 \
-    }                                                                                                                  \
-  } while (0)
-  if (dtype == PIH_F32) PIH_DELTA(float);
-  else if (dtype == PIH_BF16) PIH_DELTA(bf16);
-  else return PIH_ERR_BAD_ARGUMENT;
-#undef PIH_DELTA
+// b [rows, ldb]: write-strength logits a head; a [rows, lda] (a_dtype): decay logits, one a head or (channels) one a head and
+// key channel, with decay_bias of the same layout; decay_log [heads].  scratch: fp32, rows * (2 * kv_heads * dim + heads +
+// heads * (channels ? dim : 1)), 16-byte aligned.  out: fp32 [rows, heads, vdim].  The state S [heads, dim, vdim] lies at the
+// start of a request's slot.
+template <typename T, int D, bool CH>
+static void launch_delta_reg(cudaStream_t s, const float* qn, const float* kn, const T* v, long long ld, const float* decay,
+                             const float* beta, float* out, float* state, long long state_stride, const int* cu_q,
+                             const int* state_slots, int requests, int heads, int kv_heads, int vdim) {
+  typedef DeltaShape<D, CH> Shape;
+  const size_t staged = 2 * static_cast<size_t>(Shape::kChunk) *
+                        (Shape::kVecs * Shape::kParts * Shape::kSeg + 4 + 32 * sizeof(T) / 4) * sizeof(float);
+  if (staged > 48 * 1024)
+    cudaFuncSetAttribute(delta_recurrence_reg_kernel<T, D, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                         static_cast<int>(staged));
+  launch_kernel(delta_recurrence_reg_kernel<T, D, CH>, dim3(requests, heads, (vdim + 31) / 32), dim3(Shape::kThreads), staged, s,
+                qn, kn, v, ld, decay, beta, out, state, state_stride, cu_q, state_slots, heads, kv_heads, vdim);
+}
+
+template <typename T, bool CH>
+static int launch_delta(cudaStream_t s, const float* qn, const float* kn, const T* v, long long ld, const float* decay,
+                        const float* beta, float* out, float* state, long long state_stride, const int* cu_q,
+                        const int* state_slots, int requests, int heads, int kv_heads, int dim, int vdim) {
+  const bool words = sizeof(T) == 4 || (ld % 2 == 0 && vdim % 2 == 0 && (reinterpret_cast<uintptr_t>(v) & 3) == 0);
+  switch (words ? dim : 0) {                                   // (values are copied in 32-bit words)
+#define PIH_DELTA_REG(D)                                                                                               \
+  case D:                                                                                                              \
+    launch_delta_reg<T, D, CH>(s, qn, kn, v, ld, decay, beta, out, state, state_stride, cu_q, state_slots, requests,   \
+                               heads, kv_heads, vdim);                                                                 \
+    break
+    PIH_DELTA_REG(16);
+    PIH_DELTA_REG(32);
+    PIH_DELTA_REG(64);
+    PIH_DELTA_REG(128);
+    PIH_DELTA_REG(256);
 #undef PIH_DELTA_REG
+    default: {
+      const int cols = vdim >= 64 ? 64 : 32;
+      if (dim > 8 * cols) return PIH_ERR_UNSUPPORTED;
+      const size_t smem = (static_cast<size_t>(dim) * cols + 2 * (CH ? 3 : 2) * static_cast<size_t>(dim)) * sizeof(float);
+      if (smem > 200 * 1024) return PIH_ERR_UNSUPPORTED;
+      if (smem > 48 * 1024)
+        cudaFuncSetAttribute(delta_recurrence_kernel<T, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             static_cast<int>(smem));
+      const dim3 grid(requests, heads, (vdim + cols - 1) / cols);
+      launch_kernel(delta_recurrence_kernel<T, CH>, grid, dim3(cols), smem, s, qn, kn, v, ld, decay, beta, out, state,
+                    state_stride, cu_q, state_slots, heads, kv_heads, dim, vdim);
+    }
+  }
   PIH_LAUNCH_CHECK();
   return 0;
 }
 
-extern "C" int pih_gated_rmsnorm(int dtype, const void* o, const void* gate, long long ldg, const void* weight, void* out,
-                                 int rows, int heads, int vdim, float eps, void* stream) {
+extern "C" int pih_gated_delta_rule(int dtype, const void* qkv, long long ld, const void* b, long long ldb, int a_dtype,
+                                    const void* a, long long lda, int channels, const void* decay_log,
+                                    const void* decay_bias, void* scratch, void* out, void* state, long long state_stride,
+                                    const void* cu_q, const void* state_slots, int rows, int requests, int heads,
+                                    int kv_heads, int dim, int vdim, float unit_eps, float q_scale, void* stream) {
+  if (rows <= 0 || requests <= 0) return 0;
+  if (heads % kv_heads) return PIH_ERR_BAD_ARGUMENT;
+  if (heads > 65535 || (vdim + 31) / 32 > 65535) return PIH_ERR_UNSUPPORTED;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const long long qk_size = static_cast<long long>(kv_heads) * dim;
+  float* qn = static_cast<float*>(scratch);
+  float* kn = qn + rows * qk_size;
+  float* decay = kn + rows * qk_size;
+  float* beta = decay + static_cast<long long>(rows) * heads * (channels ? dim : 1);
+#define PIH_DELTA(T, TA)                                                                                               \
+  do {                                                                                                                 \
+    launch_kernel(delta_prepare_kernel<T, TA>, dim3(rows), dim3(128), 0, s, static_cast<const T*>(qkv), ld,            \
+                  static_cast<const T*>(b), ldb, static_cast<const TA*>(a), lda, channels,                             \
+                  static_cast<const float*>(decay_log), static_cast<const float*>(decay_bias), qn, kn, decay, beta,    \
+                  heads, kv_heads, dim, unit_eps, q_scale);                                                            \
+    PIH_LAUNCH_CHECK();                                                                                                \
+    const T* v = static_cast<const T*>(qkv) + 2 * qk_size;                                                             \
+    float* o = static_cast<float*>(out);                                                                               \
+    float* st = static_cast<float*>(state);                                                                            \
+    const int* cu = static_cast<const int*>(cu_q);                                                                     \
+    const int* slots = static_cast<const int*>(state_slots);                                                           \
+    return channels ? launch_delta<T, true>(s, qn, kn, v, ld, decay, beta, o, st, state_stride, cu, slots, requests,   \
+                                            heads, kv_heads, dim, vdim)                                                \
+                    : launch_delta<T, false>(s, qn, kn, v, ld, decay, beta, o, st, state_stride, cu, slots, requests,  \
+                                             heads, kv_heads, dim, vdim);                                              \
+  } while (0)
+  if (dtype == PIH_F32 && a_dtype == PIH_F32) PIH_DELTA(float, float);
+  if (dtype == PIH_BF16 && a_dtype == PIH_BF16) PIH_DELTA(bf16, bf16);
+  if (dtype == PIH_BF16 && a_dtype == PIH_F32) PIH_DELTA(bf16, float);
+  return PIH_ERR_BAD_ARGUMENT;
+#undef PIH_DELTA
+}
+
+// o fp32 [rows, heads, vdim]; gate [rows, ldg] (gate_dtype), out [rows, ldo] (dtype); activation 0: SiLU, 1: sigmoid.
+extern "C" int pih_gated_rmsnorm(int dtype, int gate_dtype, const void* o, const void* gate, long long ldg,
+                                 const void* weight, void* out, long long ldo, int rows, int heads, int vdim, float eps,
+                                 int activation, float out_scale, void* stream) {
   if (rows <= 0) return 0;
+  if (activation < 0 || activation > 1) return PIH_ERR_BAD_ARGUMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const long long items = static_cast<long long>(rows) * heads;
   dim3 grid(static_cast<unsigned>((items + 3) / 4));
-#define PIH_GN(T)                                                                                                      \
-  launch_kernel(gated_rmsnorm_kernel<T>, grid, dim3(128), 0, s, static_cast<const float*>(o), static_cast<const T*>(gate), \
-                ldg, static_cast<const float*>(weight), static_cast<T*>(out), items, heads, vdim, eps)
-  if (dtype == PIH_F32) PIH_GN(float);
-  else if (dtype == PIH_BF16) PIH_GN(bf16);
+#define PIH_GN(TG, T)                                                                                                  \
+  launch_kernel(gated_rmsnorm_kernel<TG, T>, grid, dim3(128), 0, s, static_cast<const float*>(o), static_cast<const TG*>(gate), \
+                ldg, static_cast<const float*>(weight), static_cast<T*>(out), ldo, items, heads, vdim, eps, activation, out_scale)
+  if (dtype == PIH_F32 && gate_dtype == PIH_F32) PIH_GN(float, float);
+  else if (dtype == PIH_BF16 && gate_dtype == PIH_BF16) PIH_GN(bf16, bf16);
+  else if (dtype == PIH_BF16 && gate_dtype == PIH_F32) PIH_GN(float, bf16);
   else return PIH_ERR_BAD_ARGUMENT;
 #undef PIH_GN
   PIH_LAUNCH_CHECK();

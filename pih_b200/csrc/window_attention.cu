@@ -1,12 +1,13 @@
-// Softmax attention over a sliding window with optional kept first tokens, a sink in the denominator, a learned bias
-// by distance, capped scores and a gate a head.
+// Softmax attention over a sliding window or inside chunks of places, with optional kept first tokens, a sink in the
+// denominator, a learned bias by distance, capped scores and a gate a head.
 //
 // The cache holds one vector per token, [k: kv_heads x dim | v: kv_heads x vdim], in pages: cache[page][offset][width].
-// A row at position p sees the keys j <= p with p - j < window (window 0: all) or j < keep_first.
+// A row at position p sees the keys j <= p with p - j < window (window 0: all) and j / chunk == p / chunk (chunk 0: all;
+// chunks count from place 0 of the sequence), or j < keep_first.
 //
 //   score  = (q . k) scale;  cap > 0: cap tanh(score / cap);  bias: + bias[head][min(p - j, distances - 1)]
 //   weight = exp(score) / (sum over the seen keys of exp(score) + exp(sink[head]))        (sink null: no such term)
-//   out    = sum weight v, times sigmoid(gate[row][head]) where there is a gate
+//   out    = sum weight v, times sigmoid(gate[row][head]) where there is a gate, times one number
 //
 //   window_qk_prepare        per row: RMS norm over the WHOLE q (and k) projection with a weight a column, rotation of the
 //                            first columns of every head in neighbouring pairs or in halves, by a table of (cos, sin) or
@@ -33,11 +34,19 @@ constexpr int kWinMaxPerLane = 16;          // value columns a lane at most: vdi
 // What a row may see, and how a score is finished: shared by all kernels of the file.
 struct WindowRule {
   int window;            // 0: every earlier key
+  int chunk;             // 0: none; only keys of the row's own chunk of this many places
   int keep_first;        // keys below this place stay seen
   float scale;
   float cap;             // 0: scores are not capped
   const float* bias;     // [heads][distances] or null
   int distances;
+  float out_scale;       // multiplies the output
+  // the first key that a row at ``pos`` sees (apart from the kept ones); grows with ``pos``
+  __device__ __forceinline__ int first_of(int pos) const {
+    int first = window > 0 ? max(0, pos - window + 1) : 0;
+    if (chunk > 0 && pos > 0) first = max(first, pos - pos % chunk);
+    return first;
+  }
 };
 
 template <bool kExact>
@@ -349,7 +358,8 @@ __device__ __forceinline__ void window_stretch(const float* q, const T* __restri
 // The sink joins the denominator, the sums are divided, the gate multiplies; a lane holds columns PL lane + e.
 template <typename T, int PL>
 __device__ __forceinline__ void window_finish(float (&a)[PL], float m, float l, const float* __restrict__ sink, int head,
-                                              const T* __restrict__ gate, int vdim, int lane, T* __restrict__ out,
+                                              const T* __restrict__ gate, float scale, int vdim, int lane,
+                                              T* __restrict__ out,
                                               uint32_t* __restrict__ error) {
   float fix = 1.0f;
   if (sink != nullptr) {
@@ -362,7 +372,7 @@ __device__ __forceinline__ void window_finish(float (&a)[PL], float m, float l, 
     if (lane == 0) publish_error(error, kAttentionDenominator);
     l = 1.0f;
   }
-  float f = fix / l;
+  float f = fix / l * scale;
   if (gate != nullptr) f *= 1.0f / (1.0f + expf(-to_float<T>(*gate)));
 #pragma unroll
   for (int e = 0; e < PL; ++e)
@@ -373,7 +383,7 @@ __device__ __forceinline__ void window_finish(float (&a)[PL], float m, float l, 
 // keys of rows whose request brings at most small_rows rows, its sums to partial [row][head][split][2 + 32 PL]: m, l, a (lane by lane).
 template <typename T, int PL>
 __global__ void __launch_bounds__(128)
-window_attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* __restrict__ cache,
+window_attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, long long ldo, const T* __restrict__ cache,
                                 const int* __restrict__ block_table, int table_width,
                                 const int* __restrict__ request_of_row, const int* __restrict__ positions,
                                 const int* __restrict__ cu_q, int rows, int heads, int kv_heads, int dim, int vdim,
@@ -388,7 +398,7 @@ window_attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, co
   if (unit >= static_cast<long long>(rows) * heads) return;
   const int row = static_cast<int>(unit / heads), head = static_cast<int>(unit % heads);
   const int req = request_of_row[row];
-  T* o = out + unit * vdim;
+  T* o = out + row * ldo + static_cast<long long>(head) * vdim;
   if (req < 0) {                                               // a row of padding: zeros, so that nothing unset travels on
     if (blockIdx.y == 0)
       for (int e = lane; e < vdim; e += 32) o[e] = from_float<T>(0.0f);
@@ -401,7 +411,7 @@ window_attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, co
   for (int e = lane; e < dim; e += 32) qs[e] = to_float<T>(qr[e]);
   __syncwarp();
   const int pos = positions[row];
-  const int first = rule.window > 0 ? max(0, pos - rule.window + 1) : 0;
+  const int first = rule.first_of(pos);
   const int kept = min(rule.keep_first, first);                // keys 0 .. kept - 1 lie before the window and stay seen
   const int* table = block_table + static_cast<long long>(req) * table_width;
   const float* bias_of_head = rule.bias != nullptr ? rule.bias + static_cast<long long>(head) * rule.distances : nullptr;
@@ -439,14 +449,16 @@ window_attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, co
       p[2 + 32 * e + lane] = a[e];                             // (column PL lane + e; beyond vdim: zero)
     return;
   }
-  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head : nullptr, vdim, lane, o, error);
+  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head : nullptr, rule.out_scale, vdim, lane,
+                       o, error);
 }
 
 // A warp a (row, head): the parts' sums folded in order, then the sink, the division and the gate.
 template <typename T, int PL>
 __global__ void __launch_bounds__(128)
-window_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, const int* __restrict__ request_of_row,
-                              const int* __restrict__ cu_q, int rows, int heads, int vdim, int splits, int small_rows,
+window_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, long long ldo,
+                              const int* __restrict__ request_of_row, const int* __restrict__ cu_q, int rows, int heads,
+                              int vdim, int splits, int small_rows, float out_scale,
                               const float* __restrict__ sink, const T* __restrict__ gate, long long ld_gate,
                               uint32_t* __restrict__ error) {
   wait_for_prior_kernels();
@@ -477,8 +489,8 @@ window_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
     for (int e = 0; e < PL; ++e)
       a[e] = fmaf(p[2 + 32 * e + lane], d, a[e]);
   }
-  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head : nullptr, vdim, lane,
-                       out + unit * vdim, error);
+  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head : nullptr, out_scale, vdim, lane,
+                       out + row * ldo + static_cast<long long>(head) * vdim, error);
 }
 
 // Tensor cores for requests of more than small_rows rows (bf16).  A block is kTileRows consecutive rows of one request and one
@@ -493,7 +505,7 @@ constexpr int kTileRows = 16 * kTileWarps, kTileThreads = 32 * kTileWarps;
 
 template <int DIM, int VDIM>
 __global__ void __launch_bounds__(kTileThreads, 2)
-window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out,
+window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, long long ldo,
                              const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table, int table_width,
                              const int* __restrict__ cu_q, const int* __restrict__ q_start, int requests, int heads,
                              int kv_heads, int dim, int vdim, int page_size, int num_pages, WindowRule rule,
@@ -535,8 +547,8 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
   const long long width = static_cast<long long>(kv_heads) * (dim + vdim);
   const int* table = block_table + static_cast<long long>(req) * table_width;
   const int key_last = pos0 + nrows - 1;
-  const int key_first = rule.window > 0 ? max(0, pos0 - rule.window + 1) : 0;
-  const int kept = min(rule.keep_first, key_first);           // kept keys that lie before the first row's window
+  const int key_first = rule.first_of(pos0);
+  const int kept = min(rule.keep_first, key_first);           // kept keys that lie before the first row's first key
   const float* bias_of_head = rule.bias != nullptr ? rule.bias + static_cast<long long>(head) * rule.distances : nullptr;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   const int page_shift = (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;
@@ -589,6 +601,8 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
   const int ra = wr0 + (lane >> 2), rb = ra + 8;
   const int pos_a = ra < nrows ? pos0 + ra : -1, pos_b = rb < nrows ? pos0 + rb : -1;
   const int warp_first = pos0 + wr0, warp_last = pos0 + min(wr0 + 15, nrows - 1);
+  const int first_a = rule.first_of(pos_a), first_b = rule.first_of(pos_b);                // of the thread's two rows
+  const int first_low = rule.first_of(warp_first), first_high = rule.first_of(warp_last);  // of the warp's first and last
   const bool plain = rule.cap <= 0.0f && bias_of_head == nullptr;
   float O[VDIM / 8][4];
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
@@ -601,7 +615,7 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
     const int j0 = tile_of(v) * 64;
     // the warp's rows see something of this tile: a key of their windows, or a kept key
     const bool any = wr0 < nrows && j0 <= warp_last &&
-                     (rule.window <= 0 || j0 + 63 > warp_first - rule.window || j0 < rule.keep_first);
+                     (j0 + 63 >= first_low || j0 < rule.keep_first);
     const bf16* kb = Ks + buf * 64 * QLD;
     const bf16* vb = Vs + buf * 64 * VLD;
     float S[8][4];
@@ -634,7 +648,7 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
     if (v + 1 < visits) load_keys(buf ^ 1, tile_of(v + 1) * 64);
     if (any) {
       // a tile that every row of the warp sees whole needs no mask
-      const bool whole = j0 + 63 <= warp_first && (rule.window <= 0 || j0 > warp_last - rule.window || j0 + 63 < rule.keep_first);
+      const bool whole = j0 + 63 <= warp_first && (j0 >= first_high || j0 + 63 < rule.keep_first);
       const float* bias_t = bias_of_head != nullptr ? bias_s[buf] + 63 : nullptr;
       const int la = ra - 2 * (lane & 3), lb = rb - 2 * (lane & 3);   // row - key of the thread's first column
       float top_a = -INFINITY, top_b = -INFINITY;
@@ -666,8 +680,8 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
             const int key = j0 + n * 8 + 2 * (lane & 3) + c;
-            const bool see_a = key <= pos_a && (rule.window <= 0 || key > pos_a - rule.window || key < rule.keep_first);
-            const bool see_b = key <= pos_b && (rule.window <= 0 || key > pos_b - rule.window || key < rule.keep_first);
+            const bool see_a = key <= pos_a && (key >= first_a || key < rule.keep_first);
+            const bool see_b = key <= pos_b && (key >= first_b || key < rule.keep_first);
             const float sa = plain ? S[n][c] * (rule.scale * kLog2e) : finish(S[n][c], la - n * 8 - c);
             const float sb = plain ? S[n][2 + c] * (rule.scale * kLog2e) : finish(S[n][2 + c], lb - n * 8 - c);
             S[n][c] = see_a ? sa : -INFINITY;
@@ -767,7 +781,7 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
   }
   const bool bad = (ra < nrows && (!(l_a > 0.0f) || l_a > 3.0e38f)) || (rb < nrows && (!(l_b > 0.0f) || l_b > 3.0e38f));
   if (bad) publish_error(error, kAttentionDenominator);
-  float f_a = l_a > 0.0f ? fix_a / l_a : 0.0f, f_b = l_b > 0.0f ? fix_b / l_b : 0.0f;
+  float f_a = l_a > 0.0f ? fix_a / l_a * rule.out_scale : 0.0f, f_b = l_b > 0.0f ? fix_b / l_b * rule.out_scale : 0.0f;
   if (gate != nullptr) {
     if (ra < nrows) f_a *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(row0 + ra) * ld_gate + head])));
     if (rb < nrows) f_b *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(row0 + rb) * ld_gate + head])));
@@ -777,10 +791,10 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
     const int col = n * 8 + 2 * (lane & 3);
     if (col >= vdim) continue;                                // vdim is a multiple of 8: the pair is inside
     if (ra < nrows)
-      *reinterpret_cast<__nv_bfloat162*>(out + (static_cast<long long>(row0 + ra) * heads + head) * vdim + col) =
+      *reinterpret_cast<__nv_bfloat162*>(out + (row0 + ra) * ldo + static_cast<long long>(head) * vdim + col) =
           __floats2bfloat162_rn(O[n][0] * f_a, O[n][1] * f_a);
     if (rb < nrows)
-      *reinterpret_cast<__nv_bfloat162*>(out + (static_cast<long long>(row0 + rb) * heads + head) * vdim + col) =
+      *reinterpret_cast<__nv_bfloat162*>(out + (row0 + rb) * ldo + static_cast<long long>(head) * vdim + col) =
           __floats2bfloat162_rn(O[n][2] * f_b, O[n][3] * f_b);
   }
 }
@@ -824,7 +838,7 @@ extern "C" int pih_window_qk_prepare(int dtype, const void* src, long long ld, v
 }
 
 template <int DIM, int VDIM>
-static int launch_window_tile(cudaStream_t s, unsigned tiles, const void* q, void* out, const void* cache,
+static int launch_window_tile(cudaStream_t s, unsigned tiles, const void* q, void* out, long long ldo, const void* cache,
                               const void* block_table, int table_width, const void* cu_q, const void* q_start, int requests,
                               int heads, int kv_heads, int dim, int vdim, int page_size, int num_pages, const WindowRule& rule,
                               const void* sink, const void* gate, long long ld_gate, int small_rows, void* error) {
@@ -836,7 +850,7 @@ static int launch_window_tile(cudaStream_t s, unsigned tiles, const void* q, voi
     raised = true;
   }
   launch_kernel(window_attention_tile_kernel<DIM, VDIM>, dim3(tiles, heads), dim3(kTileThreads), smem, s, static_cast<const bf16*>(q),
-                static_cast<bf16*>(out), static_cast<const bf16*>(cache), static_cast<const int*>(block_table), table_width,
+                static_cast<bf16*>(out), ldo, static_cast<const bf16*>(cache), static_cast<const int*>(block_table), table_width,
                 static_cast<const int*>(cu_q), static_cast<const int*>(q_start), requests, heads, kv_heads, dim, vdim,
                 page_size, num_pages, rule, static_cast<const float*>(sink), static_cast<const bf16*>(gate), ld_gate,
                 small_rows, static_cast<uint32_t*>(error));
@@ -849,26 +863,30 @@ extern "C" int pih_window_attention_tile_takes(int dim, int vdim) {
   return dim >= 8 && vdim >= 8 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 128 && vdim <= 128;
 }
 
-// The attention of the step's rows: q [rows, heads x dim] (prepared), out [rows, heads x vdim].  bias fp32
+// The attention of the step's rows: q [rows, heads x dim] (prepared), out [rows, ldo] (heads x vdim columns are written,
+// times out_scale).  bias fp32
 // [heads, distances] or null; sink fp32 [heads] or null; gate [rows, ld_gate] of the compute dtype (column h: head h's
 // logit) or null.  ``tile`` (bf16 only, sizes that pih_window_attention_tile_takes): requests of more than 16 rows run
 // on the tensor-core kernel.  ``small``: the other rows (all rows without ``tile``) run on the warp kernel, their keys
 // cut into ``splits`` parts (1: uncut) through ``partial`` (fp32 [rows, heads, splits, 2 + 32 x the value columns a lane]).
-extern "C" int pih_window_attention(int dtype, const void* q, void* out, const void* cache, const void* block_table,
-                                    int table_width, const void* request_of_row, const void* positions, const void* cu_q,
+extern "C" int pih_window_attention(int dtype, const void* q, void* out, long long ldo, float out_scale,
+                                    const void* cache, const void* block_table, int table_width, const void* request_of_row, const void* positions, const void* cu_q,
                                     const void* q_start, int rows, int requests, int heads, int kv_heads, int dim, int vdim,
                                     int page_size, int num_pages, float scale, float cap, const void* bias, int distances,
-                                    int window, int keep_first, const void* sink, const void* gate, long long ld_gate,
+                                    int window, int chunk, int keep_first, const void* sink, const void* gate, long long ld_gate,
                                     int tile, int small, int splits, void* partial, void* error, void* stream) {
   if (rows <= 0) return 0;
   if (dim > 1024 || vdim > 32 * kWinMaxPerLane || heads % kv_heads || splits < 1) return PIH_ERR_UNSUPPORTED;
-  if (tile && (dtype != PIH_BF16 || !pih_window_attention_tile_takes(dim, vdim))) return PIH_ERR_UNSUPPORTED;
-  if (splits > 32 || (splits > 1 && partial == nullptr) || window < 0 || keep_first < 0 || (bias != nullptr && distances < 1))
+  if (tile && (dtype != PIH_BF16 || !pih_window_attention_tile_takes(dim, vdim) || ldo % 2)) return PIH_ERR_UNSUPPORTED;
+  if (ldo < static_cast<long long>(heads) * vdim) return PIH_ERR_BAD_ARGUMENT;
+  if (splits > 32 || (splits > 1 && partial == nullptr) || window < 0 || chunk < 0 || keep_first < 0 || (bias != nullptr && distances < 1))
     return PIH_ERR_BAD_ARGUMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   WindowRule rule;
   rule.window = window;
-  rule.keep_first = window > 0 ? keep_first : 0;
+  rule.chunk = chunk;
+  rule.keep_first = window > 0 || chunk > 0 ? keep_first : 0;
+  rule.out_scale = out_scale;
   rule.scale = scale;
   rule.cap = cap;
   rule.bias = static_cast<const float*>(bias);
@@ -878,7 +896,7 @@ extern "C" int pih_window_attention(int dtype, const void* q, void* out, const v
     const unsigned tiles = static_cast<unsigned>((rows + kTileRows - 1) / kTileRows + requests);
     int rc;
 #define PIH_TILE(D, V)                                                                                                 \
-  rc = launch_window_tile<D, V>(s, tiles, q, out, cache, block_table, table_width, cu_q, q_start, requests, heads,    \
+  rc = launch_window_tile<D, V>(s, tiles, q, out, ldo, cache, block_table, table_width, cu_q, q_start, requests, heads,    \
                                 kv_heads, dim, vdim, page_size, num_pages, rule, sink, gate, ld_gate, small_rows, error)
     if (dim <= 32) { if (vdim <= 64) PIH_TILE(32, 64); else PIH_TILE(32, 128); }
     else if (dim <= 64) { if (vdim <= 64) PIH_TILE(64, 64); else PIH_TILE(64, 128); }
@@ -893,7 +911,7 @@ extern "C" int pih_window_attention(int dtype, const void* q, void* out, const v
 #define PIH_WAG_PL(T, PL)                                                                                              \
   do {                                                                                                                 \
     launch_kernel(window_attention_generic_kernel<T, PL>, grid, dim3(128), smem, s, static_cast<const T*>(q),          \
-                  static_cast<T*>(out), static_cast<const T*>(cache), static_cast<const int*>(block_table), table_width, \
+                  static_cast<T*>(out), ldo, static_cast<const T*>(cache), static_cast<const int*>(block_table), table_width, \
                   static_cast<const int*>(request_of_row), static_cast<const int*>(positions),                         \
                   static_cast<const int*>(cu_q), rows, heads, kv_heads, dim, vdim, page_size, num_pages, rule,         \
                   static_cast<const float*>(sink), static_cast<const T*>(gate), ld_gate, splits, small_rows,           \
@@ -901,8 +919,8 @@ extern "C" int pih_window_attention(int dtype, const void* q, void* out, const v
     PIH_LAUNCH_CHECK();                                                                                                \
     if (splits > 1)                                                                                                    \
       launch_kernel(window_attention_merge_kernel<T, PL>, dim3(grid.x), dim3(128), 0, s,                               \
-                    static_cast<const float*>(partial), static_cast<T*>(out), static_cast<const int*>(request_of_row), \
-                    static_cast<const int*>(cu_q), rows, heads, vdim, splits, small_rows,                              \
+                    static_cast<const float*>(partial), static_cast<T*>(out), ldo, static_cast<const int*>(request_of_row), \
+                    static_cast<const int*>(cu_q), rows, heads, vdim, splits, small_rows, rule.out_scale,              \
                     static_cast<const float*>(sink), static_cast<const T*>(gate), ld_gate, static_cast<uint32_t*>(error)); \
   } while (0)
 #define PIH_WAG(T)                                                                                                     \

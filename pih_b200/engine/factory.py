@@ -1,6 +1,7 @@
 """Puts a model folder, the kernels, a cache and the step function together."""
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -52,16 +53,27 @@ def cache_tokens_for_memory(model, *, page_size: int, max_requests: int, max_bat
     esize = torch.empty((), dtype=rt.dtype).element_size()
     per_token = 0
     widest = 4 * spec.hidden
+    states = 0
     for entry, need in zip(spec.schedule, model.cache_needs()):
+        state = getattr(need, "state", need)                       # (pages and a state: both)
+        need = getattr(need, "paged", need)
         if hasattr(need, "kv_heads"):
             per_token += 2 * need.kv_heads * need.head_dim * esize
         elif hasattr(need, "width"):                               # one cached vector per token
             per_token += need.width * esize
+        if hasattr(state, "shape"):                                # a state slot a request, and its copy before a step
+            states += 2 * math.prod(state.shape) * torch.empty((), dtype=state.dtype).element_size()
+
+    def mixer_numbers(m) -> int:
+        if hasattr(m, "left"):                                     # two mixers side by side
+            return mixer_numbers(m.left) + mixer_numbers(m.right)
+        numbers = {"q_size": 2, "kv_size": 3, "qk_size": 6, "v_size": 6, "inner": 6, "decays": 2}
+        return sum(times * getattr(m, name, 0) for name, times in numbers.items())
+
     for block in spec.blocks:
         mixer, ffn = block.mixer, block.ffn
-        widest = max(widest, 4 * spec.hidden + 2 * getattr(mixer, "q_size", 0) + 3 * getattr(mixer, "kv_size", 0)
-                     + 3 * getattr(ffn, "intermediate", 0))
-    workspace = max_batch_tokens * widest * esize + 6 * max_requests * spec.vocab * 4 + (768 << 20)
+        widest = max(widest, 4 * spec.hidden + mixer_numbers(mixer) + 3 * getattr(ffn, "intermediate", 0))
+    workspace = max_batch_tokens * widest * esize + 6 * max_requests * spec.vocab * 4 + max_requests * states + (768 << 20)
     budget = int(free - (1.0 - memory_fraction) * total - workspace)
     wanted = max_requests * (-(-max_context // page_size) * page_size)
     tokens = wanted if per_token == 0 else min(wanted, budget // per_token // page_size * page_size)

@@ -112,7 +112,7 @@ class CudaOps:
                      "pih_diff_qk_prepare", "pih_diff_attention", "pih_diff_attention_tile_takes", "pih_moe_route_scored",
                      "pih_act_mul", "pih_embed_positions", "pih_hyper_stream", "pih_window_qk_prepare",
                      "pih_window_attention", "pih_window_attention_tile_takes", "pih_embed_bigram", "pih_rmsnorm_rows",
-                     "pih_rotate_heads", "pih_gate_mul", "pih_unary_act", "pih_scale_rows", "pih_moe_gather_scaled"):
+                     "pih_rotate_heads", "pih_gate_mul", "pih_unary_act", "pih_selective_scan", "pih_gemm_skinny_bias_gelu", "pih_scale_rows", "pih_moe_gather_scaled"):
             getattr(lib, name).restype = c_int
         lib.pih_attention_scratch_floats.restype = c_ll
         lib.pih_top_logprobs_scratch_words.restype = c_ll
@@ -194,14 +194,16 @@ class CudaOps:
         return c_void_p(self._error.data_ptr())
 
     # -- ops ----------------------------------------------------------------------
-    def embedding(self, table: torch.Tensor, ids: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    def embedding(self, table: torch.Tensor, ids: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
+                  scale: float = 1.0) -> torch.Tensor:
+        """``table[ids] * scale``; a scale other than 1 gives 32-bit rows (the product is not rounded again)."""
         rows, (vocab, hidden) = ids.shape[0], table.shape
-        if out_dtype is not None and out_dtype != table.dtype:
-            if out_dtype != torch.float32:
-                raise ValueError("an embedding widens to float32 only")
+        if (out_dtype is not None and out_dtype != table.dtype) or scale != 1.0:
+            if (out_dtype or table.dtype) != torch.float32:
+                raise ValueError("an embedding widens to float32 only, and only such a one is scaled")
             out = torch.empty(rows, hidden, dtype=torch.float32, device=table.device)      # a 32-bit residual stream
             rc = self.lib.pih_embedding_stream(_DT[table.dtype], _ptr(table), _ptr(ids), _ptr(out), rows, hidden, vocab,
-                                               self._err(), self._stream())
+                                               c_float(scale), self._err(), self._stream())
             self._check(rc, "embedding_stream")
             return out
         out = torch.empty(rows, hidden, dtype=table.dtype, device=table.device)
@@ -620,15 +622,27 @@ class CudaOps:
 
     # -- a residual stream in 32-bit, mixers with state, attention over a latent, routed experts ------------------
     def rmsnorm_stream(self, h: torch.Tensor, weight: torch.Tensor, eps: float, delta: Optional[torch.Tensor] = None,
-                       rows: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
-        """RMS norm of a 32-bit stream: ``h += delta`` in 32-bit (stored back unless ``rows`` selects), then
-        ``h / sqrt(mean(h^2) + eps) * weight`` rounded to ``out_dtype``.  ``weight``: fp32, one number or one a column."""
+                       rows: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.bfloat16, scale: float = 1.0,
+                       bias: Optional[torch.Tensor] = None, again: Optional[tuple] = None,
+                       vector: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """RMS norm of a 32-bit stream: ``h += scale * (delta + bias)`` in 32-bit (stored back unless ``rows`` selects),
+        then ``h / sqrt(mean(h^2) + eps) * weight`` rounded to ``out_dtype``.  ``weight``: fp32, one number or one a
+        column; ``bias``: fp32 ``[width]``, with a delta only.  Before the norm, where they are given: ``again`` = (table,
+        ids, factor): ``h += factor * table[ids]``; ``vector`` (fp32 ``[width]``): ``h += vector``."""
         width = h.shape[-1]
         assert h.dtype == torch.float32 and h.is_contiguous() and weight.dtype == torch.float32
         assert delta is None or (delta.is_contiguous() and delta.shape == h.shape)
+        assert bias is None or (delta is not None and bias.dtype == torch.float32 and bias.shape == (width,))
+        assert vector is None or (vector.dtype == torch.float32 and vector.is_contiguous() and vector.shape == (width,))
+        table, ids, factor = again if again is not None else (None, None, 0.0)
+        assert table is None or (table.is_contiguous() and table.shape[1] == width and ids.dtype == torch.int32
+                                 and (delta is None or delta.dtype == table.dtype))
+        added = delta if delta is not None else table
         n_out = h.numel() // width if rows is None else rows.shape[0]
         out = torch.empty((n_out, width), dtype=out_dtype, device=h.device)
-        rc = self.lib.pih_rmsnorm_stream(_DT[delta.dtype] if delta is not None else 0, _DT[out_dtype], _ptr(h), _ptr(delta),
+        rc = self.lib.pih_rmsnorm_stream(_DT[added.dtype] if added is not None else 0, _DT[out_dtype], _ptr(h), _ptr(delta),
+                                         c_float(scale), _ptr(bias), _ptr(table), _ptr(ids),
+                                         table.shape[0] if table is not None else 0, c_float(factor), _ptr(vector),
                                          _ptr(weight), weight.numel(), _ptr(out), _ptr(rows), n_out, width, c_float(eps),
                                          self._stream())
         self._check(rc, "rmsnorm_stream")
@@ -704,18 +718,24 @@ class CudaOps:
         self.launches += 1 if taps > 1 else 0                  # (the history's kernel)
         return out
 
-    def gated_delta_rule(self, qkv: torch.Tensor, ba: torch.Tensor, *, decay_log, decay_bias, state: torch.Tensor, step,
-                         heads: int, kv_heads: int, key_dim: int, value_dim: int, unit_eps: float,
-                         q_scale: float) -> torch.Tensor:
+    def gated_delta_rule(self, qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, *, decay_log, decay_bias,
+                         state: torch.Tensor, step, heads: int, kv_heads: int, key_dim: int, value_dim: int,
+                         unit_eps: float, q_scale: float) -> torch.Tensor:
         """The gated delta rule over the step's rows, request by request from each one's state slot
         (``state[slot, :heads * key_dim * value_dim]`` is S).  qkv ``[T, 2 kv_heads key_dim + heads value_dim]``:
-        q heads, k heads, v heads after convolution and activation; ba ``[T, 2 heads]`` (a view): write-strength
-        logits, decay logits.  Returns the read-outs, fp32 ``[T, heads, value_dim]``."""
+        q heads, k heads, v heads after convolution and activation; beta ``[T, heads]`` (a view): write-strength logits;
+        decay (a view, of the rows' dtype or fp32): decay logits, one a head ``[T, heads]`` or one a head and key channel
+        ``[T, heads * key_dim]``, with ``decay_bias`` (fp32) of the same number; ``decay_log`` fp32 ``[heads]``.  Returns
+        the read-outs, fp32 ``[T, heads, value_dim]``."""
         T = qkv.shape[0]
-        assert qkv.stride(1) == 1 and ba.stride(1) == 1 and ba.dtype == qkv.dtype
-        scratch = torch.empty(T * (2 * kv_heads * key_dim + 2 * heads), dtype=torch.float32, device=qkv.device)
+        channels = decay_bias.numel() != heads
+        per_row = heads * (key_dim if channels else 1)
+        assert qkv.stride(1) == 1 and beta.stride(1) == 1 and decay.stride(1) == 1 and beta.dtype == qkv.dtype
+        assert beta.shape[1] >= heads and decay.shape[1] >= per_row and decay_bias.numel() == per_row
+        scratch = torch.empty(T * (2 * kv_heads * key_dim + heads + per_row), dtype=torch.float32, device=qkv.device)
         out = torch.empty(T, heads, value_dim, dtype=torch.float32, device=qkv.device)
-        rc = self.lib.pih_gated_delta_rule(_DT[qkv.dtype], _ptr(qkv), c_ll(qkv.stride(0)), _ptr(ba), c_ll(ba.stride(0)),
+        rc = self.lib.pih_gated_delta_rule(_DT[qkv.dtype], _ptr(qkv), c_ll(qkv.stride(0)), _ptr(beta), c_ll(beta.stride(0)),
+                                           _DT[decay.dtype], _ptr(decay), c_ll(decay.stride(0)), 1 if channels else 0,
                                            _ptr(decay_log), _ptr(decay_bias), _ptr(scratch), _ptr(out), _ptr(state),
                                            c_ll(state.stride(0)), _ptr(step.cu_q), _ptr(step.state_slots), T,
                                            step.num_requests, heads, kv_heads, key_dim, value_dim, c_float(unit_eps),
@@ -724,15 +744,42 @@ class CudaOps:
         self.launches += 1                                     # two kernels
         return out
 
-    def gated_rmsnorm(self, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
-        """``o / sqrt(mean(o^2) + eps) * weight * silu(gate)`` per (row, head): o fp32 ``[T, heads, vdim]``, gate
-        ``[T, heads * vdim]`` (a view), weight fp32 ``[vdim]``; returns ``[T, heads * vdim]`` in the gate's dtype."""
+    def gated_rmsnorm(self, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, activation: str = "silu",
+                      scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``o / sqrt(mean(o^2) + eps) * weight * act(gate) * scale`` per (row, head): o fp32 ``[T, heads, vdim]``, gate
+        ``[T, heads * vdim]`` (a view), weight fp32 ``[vdim]``, ``activation`` "silu" or "sigmoid"; into ``out`` (a view,
+        ``[T, heads * vdim]``) or a new tensor of the gate's dtype, which is returned."""
         T, heads, vdim = o.shape
-        assert o.is_contiguous() and gate.stride(1) == 1
-        out = torch.empty(T, heads * vdim, dtype=gate.dtype, device=o.device)
-        rc = self.lib.pih_gated_rmsnorm(_DT[gate.dtype], _ptr(o), _ptr(gate), c_ll(gate.stride(0)), _ptr(weight), _ptr(out),
-                                        T, heads, vdim, c_float(eps), self._stream())
+        assert o.is_contiguous() and gate.stride(1) == 1 and gate.shape[1] >= heads * vdim
+        if out is None:
+            out = torch.empty(T, heads * vdim, dtype=gate.dtype, device=o.device)
+        assert out.shape == (T, heads * vdim) and out.stride(1) == 1
+        rc = self.lib.pih_gated_rmsnorm(_DT[out.dtype], _DT[gate.dtype], _ptr(o), _ptr(gate), c_ll(gate.stride(0)),
+                                        _ptr(weight), _ptr(out), c_ll(out.stride(0)), T, heads, vdim, c_float(eps),
+                                        {"silu": 0, "sigmoid": 1}[activation], c_float(scale), self._stream())
         self._check(rc, "gated_rmsnorm")
+        return out
+
+    def selective_scan(self, u: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, z: torch.Tensor, *, dt_bias, A, D,
+                       state: torch.Tensor, step, scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The selective scan over the step's rows from each request's state (``state[slot, :inner * n]`` is S, ``A``
+        ``[inner, n]``): ``dt = softplus(dt + dt_bias)``, ``S <- exp(dt A) S + dt u B``, ``y = S C + D u``; into ``out``
+        ``y * silu(z) * scale``.  u, z ``[T, inner]`` and bc ``[T, 2 n]`` (B, then C) of the compute dtype, dt ``[T,
+        inner]``, ``dt_bias``, ``A``, ``D`` fp32; u, z, bc, dt may be views."""
+        T, inner = u.shape
+        n = A.shape[1]
+        assert u.stride(1) == 1 and z.stride(1) == 1 and bc.stride(1) == 1 and dt.stride(1) == 1
+        assert dt.dtype == torch.float32 and bc.dtype == u.dtype == z.dtype and bc.shape[1] >= 2 * n
+        assert A.shape == (inner, n) and A.is_contiguous() and A.dtype == torch.float32 and state.dtype == torch.float32
+        if out is None:
+            out = torch.empty(T, inner, dtype=u.dtype, device=u.device)
+        assert out.dtype == u.dtype and out.shape == (T, inner) and out.stride(1) == 1
+        rc = self.lib.pih_selective_scan(_DT[u.dtype], _ptr(u), c_ll(u.stride(0)), _ptr(dt), c_ll(dt.stride(0)), _ptr(dt_bias),
+                                         _ptr(A), _ptr(bc), c_ll(bc.stride(0)), _ptr(D), _ptr(z), c_ll(z.stride(0)), _ptr(out),
+                                         c_ll(out.stride(0)), c_float(scale), _ptr(state), c_ll(state.stride(0)),
+                                         _ptr(step.cu_q), _ptr(step.state_slots), T, step.num_requests, inner, n,
+                                         self._stream())
+        self._check(rc, "selective_scan")
         return out
 
     def rglru_scan(self, u: torch.Tensor, gates: torch.Tensor, y_pre: torch.Tensor, *, y_bias, r_bias, i_bias, lam,
@@ -1104,9 +1151,11 @@ class CudaOps:
     def window_attention(self, q: torch.Tensor, *, cache: torch.Tensor, block_table: torch.Tensor, step, scale: float,
                          window: int, keep_first: int, softcap: float, bias: Optional[torch.Tensor],
                          sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], heads: int, kv_heads: int,
-                         key_dim: int, value_dim: int) -> torch.Tensor:
-        """Attention of the step's rows (q prepared, ``[T, heads x key_dim]``) over the keys of their window and the
-        kept first keys; ``bias`` fp32 ``[heads, distances]`` by distance (the last column for every larger one),
+                         key_dim: int, value_dim: int, chunk: int = 0, scale_out: float = 1.0,
+                         out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Attention of the step's rows (q prepared, ``[T, heads x key_dim]``) over the keys of their window (0: all), of
+        their chunk of ``chunk`` places (0: all; chunks count from place 0 of the sequence) and the kept first keys, into
+        ``out`` (a view) or a new tensor, times ``scale_out``; ``bias`` fp32 ``[heads, distances]`` by distance (the last column for every larger one),
         ``softcap`` 0: none, ``sink`` fp32 ``[heads]`` or None, ``gate`` ``[T, >= heads]`` (a view: column h is head
         h's logit) or None.  Returns ``[T, heads x value_dim]``.
 
@@ -1116,7 +1165,9 @@ class CudaOps:
         rows = q.shape[0]
         num_pages, page_size = cache.shape[0], cache.shape[1]
         assert q.is_contiguous() and cache.dtype == q.dtype and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1))
-        out = torch.empty(rows, heads * value_dim, dtype=q.dtype, device=q.device)
+        if out is None:
+            out = torch.empty(rows, heads * value_dim, dtype=q.dtype, device=q.device)
+        assert out.shape == (rows, heads * value_dim) and out.stride(1) == 1 and out.dtype == q.dtype
         tile, small, splits, partial = 0, 1, 1, None
         if q.dtype == torch.bfloat16 and self.window_attention_fast:
             plans = getattr(step, "attention_plans", None)
@@ -1125,23 +1176,28 @@ class CudaOps:
                 plan = self.attention_plan(step.host_cu_q, step.host_q_start, 1)
                 if plans is not None:
                     plans[1] = plan
-            if self.lib.pih_window_attention_tile_takes(key_dim, value_dim) and cache.shape[2] % 8 == 0:
+            if (self.lib.pih_window_attention_tile_takes(key_dim, value_dim) and cache.shape[2] % 8 == 0
+                    and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0):
                 tile, small = (1 if plan[0] > 0 else 0), (1 if plan[1] > 0 else 0)
             if small:
                 # a row reads at most its window and the kept keys: as many parts as bring the GPU's warps to work
                 # (32 a multiprocessor: a warp waits on its loads most of the time), and no more than leave a part
                 # 64 keys
-                reach = plan[2] if window <= 0 else min(plan[2], window + keep_first + 32)
+                reach = plan[2]
+                for bound in (window, chunk):
+                    if bound > 0:
+                        reach = min(reach, bound + keep_first + 32)
                 splits = max(1, min(32, (148 * 32) // max(1, rows * heads), max(1, reach // 64)))
                 if splits > 1:
                     per_lane = 2 if value_dim <= 64 else (4 if value_dim <= 128 else (8 if value_dim <= 256 else 16))
                     partial = torch.empty(rows * heads * splits * (2 + 32 * per_lane), dtype=torch.float32, device=q.device)
         distances = bias.shape[1] if bias is not None else 0
         rc = self.lib.pih_window_attention(
-            _DT[q.dtype], _ptr(q), _ptr(out), _ptr(cache), _ptr(block_table), block_table.shape[1],
+            _DT[q.dtype], _ptr(q), _ptr(out), c_ll(out.stride(0)), c_float(scale_out), _ptr(cache), _ptr(block_table),
+            block_table.shape[1],
             _ptr(step.request_of_row), _ptr(step.positions), _ptr(step.cu_q), _ptr(getattr(step, "q_start", None)), rows,
             step.num_requests, heads, kv_heads, key_dim, value_dim, page_size, num_pages, c_float(scale),
-            c_float(softcap or 0.0), _ptr(bias), distances, int(window), int(keep_first), _ptr(sink), _ptr(gate),
+            c_float(softcap or 0.0), _ptr(bias), distances, int(window), int(chunk), int(keep_first), _ptr(sink), _ptr(gate),
             c_ll(gate.stride(0) if gate is not None else 0), tile, small, splits, _ptr(partial), self._err(), self._stream())
         self._check(rc, "window_attention")
         self.launches += tile + (1 if splits > 1 else 0) + small - 1
@@ -1204,15 +1260,30 @@ class CudaOps:
         self._check(rc, "gate_mul")
         return out
 
-    def activation(self, z: torch.Tensor, kind: str) -> torch.Tensor:
-        """``kind`` "relu2": the square of ``max(z, 0)``; z ``[T, n]`` (rows may be strided); 32-bit inside, rounded once."""
+    def activation(self, z: torch.Tensor, kind: str, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``kind`` "relu2": the square of ``max(v, 0)``; "gelu_erf": ``v / 2 (1 + erf(v / sqrt(2)))``, with ``v = z + bias``
+        (``bias`` fp32 ``[n]`` or None); z ``[T, n]`` (rows may be strided); 32-bit inside, rounded once."""
         T, n = z.shape
-        assert z.stride(1) == 1
+        assert z.stride(1) == 1 and (bias is None or (bias.dtype == torch.float32 and bias.shape == (n,)))
         out = torch.empty(T, n, dtype=z.dtype, device=z.device)
-        rc = self.lib.pih_unary_act(_DT[z.dtype], _ptr(z), c_ll(z.stride(0)), _ptr(out), c_ll(T), n, {"relu2": 1}[kind],
-                                    self._stream())
+        rc = self.lib.pih_unary_act(_DT[z.dtype], _ptr(z), c_ll(z.stride(0)), _ptr(bias), _ptr(out), c_ll(T), n,
+                                    {"relu2": 1, "gelu_erf": 2}[kind], self._stream())
         self._check(rc, "unary_act")
         return out
+
+    def linear_bias_gelu(self, x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+        """``gelu(round(x . w^T) + bias)`` with the error-function form of GELU, rounded once more: one kernel for few
+        rows in bf16, else the product and then ``activation`` (the same values)."""
+        M, K = x.shape
+        N = w.shape[0]
+        if x.dtype == torch.bfloat16 and M <= min(self.skinny_max_rows, 16) and K % 32 == 0 and K <= 16384 and x.stride(1) == 1:
+            out = torch.empty(M, N, dtype=x.dtype, device=x.device)
+            rc = self.lib.pih_gemm_skinny_bias_gelu(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), M, N, K, c_ll(x.stride(0)),
+                                                    c_ll(w.stride(0)), c_ll(N), self._err(), self._stream())
+            if rc != -2:
+                self._check(rc, "gemm_skinny_bias_gelu")
+                return out
+        return self.activation(self.linear(x, w), "gelu_erf", bias)
 
     def scale_(self, x: torch.Tensor, scale: float) -> torch.Tensor:
         """``x *= scale`` in place; x fp32, contiguous."""

@@ -20,7 +20,7 @@ import torch
 from ..config.registry import load_config
 from ..config.specs import ModelSpec
 from ..parts import part_class
-from ..parts.registry import Runtime, StateNeed, TensorInfo
+from ..parts.registry import Pending, Runtime, StateNeed, TensorInfo
 from ..parts._bind import bind_matrix
 from ..weights.loader import load_weights, tensor_shapes
 
@@ -32,6 +32,8 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, TensorInfo]:
         out[spec.position_name] = TensorInfo((spec.max_positions, spec.hidden))
     if spec.bigram is not None:
         out[spec.bigram.name] = TensorInfo((spec.bigram.buckets + 1, spec.hidden))
+    if spec.vectors_name is not None:
+        out[spec.vectors_name] = TensorInfo((spec.vectors, spec.hidden))
     for block in spec.blocks:
         cls = part_class("block", block.arrangement)
         for rel, info in cls.expected_tensors(block).items():
@@ -55,6 +57,9 @@ class CausalLM:
         self.bigram = bind_matrix(weights[spec.bigram.name], rt) if spec.bigram is not None else None
         if self.bigram is not None and (spec.streams or self.places is not None):
             raise ValueError("a bigram embedding goes with one residual stream and no table of places")
+        self.vectors = None
+        if spec.vectors_name is not None:
+            self.vectors = weights[spec.vectors_name].to(device=rt.device, dtype=torch.float32).contiguous()
         self._ones = torch.ones(spec.streams, dtype=torch.float32, device=rt.device) if spec.streams else None
         self.blocks = []
         for block in spec.blocks:
@@ -88,6 +93,17 @@ class CausalLM:
             needs.append(StateNeed((1,), torch.int32))
         return needs
 
+    def _added(self, entry, delta, step) -> Pending:
+        """What the stream receives right before a schedule entry, behind the last sub-layer's output: the embedding
+        output once more (formed again from the table: nothing is kept of it), a vector; the entry's first norm adds all."""
+        if not isinstance(delta, Pending):
+            delta = Pending(delta)
+        if entry.add_embedding:
+            delta.again = (self.embed, step.token_ids, float(self.spec.embed_scale))
+        if entry.add_vector is not None:
+            delta.vector = self.vectors[entry.add_vector]
+        return delta
+
     # -- one pass over the rows of a step --------------------------------------
     def forward(self, step, caches) -> Optional[torch.Tensor]:
         """``step``: the packed batch; ``caches[i]``: the cache view of
@@ -109,12 +125,16 @@ class CausalLM:
         elif self.places is not None:
             h = ops.embed_positions(self.embed, self.places, step.token_ids, step.positions,
                                     out_dtype=torch.float32 if wide else self.rt.dtype).reshape(-1, self.spec.hidden)
-        elif wide:
-            h = ops.embedding(self.embed, step.token_ids, out_dtype=torch.float32)      # the residual stream stays 32-bit
+        elif wide or self.spec.embed_scale != 1.0:
+            # the residual stream stays 32-bit
+            kw = dict(scale=self.spec.embed_scale) if self.spec.embed_scale != 1.0 else {}
+            h = ops.embedding(self.embed, step.token_ids, out_dtype=torch.float32, **kw)
         else:
             h = ops.embedding(self.embed, step.token_ids)
         delta = None
         for i, entry in enumerate(self.spec.schedule):
+            if entry.add_embedding or entry.add_vector is not None:
+                delta = self._added(entry, delta, step)
             h, delta = self.blocks[entry.layer].forward(h, delta, step, caches[i])
         if step.num_logit_rows == 0:
             return None

@@ -8,12 +8,15 @@ next norm wherever that norm lives (the next block's, or the model's final
 norm).  ``delta`` is None when the last sub-layer has added its output itself
 (for few rows the output projections add the residual in their epilogue).
 A layer whose spec has no feed-forward is ``h += mixer(norm_in(h))`` alone.
+With ``residual_scale`` s the layer is ``h += s mixer(norm_in(h)); h += s
+ffn(norm_post(h))``: the factor, and a feed-forward's output bias, travel with
+the output (``Pending``) and are applied by the kernel of the next norm.
 """
 from __future__ import annotations
 
 import torch
 
-from .registry import Runtime, TensorInfo, part_class, register_block
+from .registry import Pending, Runtime, TensorInfo, part_class, register_block
 
 
 def _sub(weights, names, prefix=""):
@@ -52,6 +55,12 @@ class PreNormBlock:
                 spec.norm_post, _sub(weights, norm_post_cls.expected_tensors(spec.norm_post), n["norm_post"]), rt)
             self.ffn = ffn_cls(spec.ffn, _sub(weights, ffn_cls.expected_tensors(spec.ffn)), rt)
         self._native_ok = None             # decided at the first step
+        self._scale = float(getattr(spec, "residual_scale", 1.0))
+
+    def _pending(self, y, part):
+        """A sub-layer's output on its way to the stream: with a factor or a bias, a ``Pending`` sum."""
+        bias = getattr(part, "output_bias", None)
+        return y if self._scale == 1.0 and bias is None else Pending(y, self._scale, bias)
 
     def forward(self, h, delta, step, cache):
         # kernels that can issue a whole block of these parts from one native call get it (the same kernels in the
@@ -59,23 +68,24 @@ class PreNormBlock:
         if self._native_ok is None:
             native = getattr(self.rt.ops, "native_block", None)
             self._native_ok = native is not None and self.rt.ops._native_supports(self)
-        if self._native_ok:
+        if self._native_ok and not isinstance(delta, Pending):
             done = self.rt.ops.native_block(self, h, delta, step, cache)
             if done is not None:
                 return done
         # a part that can take "add, norm, then me" as one call gets it (fewer kernels for few rows);
         # any other part gets the normed rows
-        fused_in = getattr(self.norm_in, "fusable", False)
-        fused_post = getattr(self.norm_post, "fusable", False)
+        plain = self._scale == 1.0
+        fused_in = plain and getattr(self.norm_in, "fusable", False) and not isinstance(delta, Pending)
+        fused_post = plain and getattr(self.norm_post, "fusable", False)
         if fused_in and hasattr(self.mixer, "forward_prenorm"):
             h, a = self.mixer.forward_prenorm(h, delta, self.norm_in, step, cache)
         else:
-            a = self.mixer.forward(self.norm_in.add_forward(h, delta), step, cache)
+            a = self._pending(self.mixer.forward(self.norm_in.add_forward(h, delta), step, cache), self.mixer)
         if self.ffn is None:
             return h, a
-        if fused_post and hasattr(self.ffn, "forward_prenorm"):
+        if fused_post and hasattr(self.ffn, "forward_prenorm") and not isinstance(a, Pending):
             return self.ffn.forward_prenorm(h, a, self.norm_post)
-        return h, self.ffn.forward(self.norm_post.add_forward(h, a))
+        return h, self._pending(self.ffn.forward(self.norm_post.add_forward(h, a)), self.ffn)
 
 
 @register_block("outnorm")

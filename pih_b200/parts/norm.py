@@ -13,7 +13,7 @@ from __future__ import annotations
 
 import torch
 
-from .registry import Runtime, TensorInfo, register_norm
+from .registry import Pending, Runtime, TensorInfo, register_norm
 from ._bind import bind_vector
 
 
@@ -46,6 +46,10 @@ class RMSNorm:
         return self.add_forward(x, None, rows=rows)
 
     def add_forward(self, h, delta, rows=None):
+        if isinstance(delta, Pending):
+            return self.rt.ops.rmsnorm_stream(h, self.weight_f32, self.spec.eps, delta=delta.y, rows=rows,
+                                              out_dtype=self.rt.dtype, scale=delta.scale, bias=delta.bias, again=delta.again,
+                                              vector=delta.vector)
         if h.dtype != self.rt.dtype:
             # a residual stream kept in 32-bit beside a 16-bit compute dtype: the sum stays 32-bit, the normed rows
             # take the compute dtype
@@ -76,4 +80,8 @@ class ScalarRMSNorm:
     def add_forward(self, h, delta, rows=None):
         if h.dtype != torch.float32:
             raise TypeError("the one-number RMS norm reads a 32-bit stream")
+        if isinstance(delta, Pending):
+            return self.rt.ops.rmsnorm_stream(h, self.weight, self.spec.eps, delta=delta.y, rows=rows,
+                                              out_dtype=self.rt.dtype, scale=delta.scale, bias=delta.bias, again=delta.again,
+                                              vector=delta.vector)
         return self.rt.ops.rmsnorm_stream(h, self.weight, self.spec.eps, delta=delta, rows=rows, out_dtype=self.rt.dtype)

@@ -24,9 +24,17 @@ mixer         ``cache_need() -> PagedKVNeed | PagedVectorNeed | StateNeed | Page
               ``step`` is the engine's ``StepBatch`` (packed rows, request
               boundaries ``cu_q``, positions, state slots), ``cache`` the
               view that the cache manager made for this schedule entry.
-feed-forward  ``forward(x) -> y`` with x, y ``[T, hidden]``.
+              A mixer that is one product in front, an inner part and one
+              product behind may show them: ``w_in [n, hidden]``, ``w_o
+              [hidden, m]`` and ``inner(proj, step, cache, out=None, scale=1)``
+              from the first product's rows ``[T, n]`` (a view) to the second's
+              ``[T, m]``, written into the view ``out`` and multiplied by
+              ``scale``.  Such mixers can be run side by side (``parallel``).
+feed-forward  ``forward(x) -> y`` with x, y ``[T, hidden]``; ``output_bias``
+              (fp32 ``[hidden]``, optional): what is still to be added to y.
 block         ``forward(h, delta, step, cache) -> (h, delta)``: the residual
-              stream and the last sub-layer's output that is not added yet.
+              stream and the last sub-layer's output that is not added yet
+              (a tensor, or a ``Pending`` sum on a 32-bit stream).
 """
 from __future__ import annotations
 
@@ -54,10 +62,12 @@ class PagedKVNeed:
 class PagedVectorNeed:
     """One vector of ``width`` numbers per token (a latent that keys and values are derived from), in pages
     like keys and values: the group's tensor is ``[entries, pages, page_size, width]``.  With a ``window``, the
-    pages that hold one of the first ``keep_first`` tokens stay when the window has moved past them."""
+    pages that hold one of the first ``keep_first`` tokens stay when the window has moved past them.  With a ``chunk``,
+    only tokens of the same chunk of that many places (counted from place 0) are read again."""
     width: int
     window: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -73,6 +83,18 @@ class PagedStateNeed:
     token and also carries a few rows from step to step): the mixer's view is the paged one with ``state`` set."""
     paged: object                 # PagedKVNeed or PagedVectorNeed
     state: StateNeed
+
+
+@dataclass
+class Pending:
+    """What a 32-bit residual stream is still to receive, in this order: ``scale * (y + bias)``; ``factor * table[ids]``
+    (``again`` = (table, ids, factor): the token's embedding once more); ``vector``.  The next norm adds it in its own
+    kernel.  Absent parts are None."""
+    y: Optional[torch.Tensor] = None
+    scale: float = 1.0
+    bias: Optional[torch.Tensor] = None
+    again: Optional[tuple] = None
+    vector: Optional[torch.Tensor] = None
 
 
 @dataclass

@@ -54,12 +54,15 @@ class Retention:
         return StateNeed((s.heads * s.key_dim * s.value_dim,), torch.float32)
 
     def forward(self, x, step, cache):
+        ops = self.rt.ops
+        return ops.linear(self.inner(ops.linear(x, self.w_in), step, cache), self.w_o)
+
+    def inner(self, proj, step, cache, out=None, scale=1.0):
+        """From the rows ``[T, 2 QK + 2 VS]`` (q | k | v | gate) to what the output product reads."""
         s, ops = self.spec, self.rt.ops
         QK, VS = s.qk_size, s.v_size
-        proj = ops.linear(x, self.w_in)                                     # [T, 2 QK + 2 VS]: q | k | v | gate
         freq = self.position.frequencies() if self.position is not None else None
         o = ops.retention(proj[:, :2 * QK], proj[:, 2 * QK:2 * QK + VS], frequencies=freq,
                           decay_minus_one=self.decay_minus_one, key_scale=s.key_scale, state=cache.state, step=step,
                           heads=s.heads, key_dim=s.key_dim, value_dim=s.value_dim)
-        y = ops.gated_rmsnorm(o, proj[:, 2 * QK + VS:], self.ones, s.norm_eps)
-        return ops.linear(y, self.w_o)
+        return ops.gated_rmsnorm(o, proj[:, 2 * QK + VS:], self.ones, s.norm_eps, scale=scale, out=out)

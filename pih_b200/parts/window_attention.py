@@ -1,7 +1,7 @@
-"""Softmax attention over a sliding window with a sink in the denominator, as a mixer.
+"""Softmax attention over a sliding window or inside chunks of places, with a sink in the denominator, as a mixer.
 
-A row at position p sees the keys j <= p with ``p - j < window`` or ``j < keep_first`` (kept first keys keep their
-true positions).  With ``q [heads, key_dim]``, ``k [kv_heads, key_dim]``, ``v [kv_heads, value_dim]`` and query head h
+A row at position p sees the keys j <= p with ``p - j < window`` and (``chunk``) ``j // chunk == p // chunk``, or ``j <
+keep_first`` (kept first keys keep their true positions).  With ``q [heads, key_dim]``, ``k [kv_heads, key_dim]``, ``v [kv_heads, value_dim]`` and query head h
 reading key/value head ``h // (heads // kv_heads)``::
 
     s_j = scale q . k_j;   softcap: s_j <- c tanh(s_j / c);   bias: s_j <- s_j + rel[bucket(p - j), h]
@@ -85,8 +85,8 @@ class WindowAttention:
     def __init__(self, spec, weights, rt: Runtime):
         if spec.heads % spec.kv_heads:
             raise ValueError(f"heads ({spec.heads}) must be a multiple of kv_heads ({spec.kv_heads})")
-        if spec.window < 0 or spec.keep_first < 0:
-            raise ValueError("window and keep_first must not be negative")
+        if spec.window < 0 or spec.keep_first < 0 or spec.chunk < 0:
+            raise ValueError("window, chunk and keep_first must not be negative")
         if spec.values_from_keys and spec.value_dim != spec.key_dim:
             raise ValueError("values that are the keys need value_dim == key_dim")
         if spec.sink not in ("learned", "zero", "none"):
@@ -139,7 +139,10 @@ class WindowAttention:
         s = self.spec
         reach = getattr(s, "cache_window", None)
         reach = s.window if reach is None else reach            # (0: every key stays)
-        paged = PagedVectorNeed(s.k_size + s.v_size, reach or None, s.keep_first if reach else 0) if self.own_kv else None
+        # (a cache that another entry reads too is kept as far back as ``cache_window`` says, whatever the chunks)
+        chunk = s.chunk or None if getattr(s, "cache_window", None) is None else None
+        paged = (PagedVectorNeed(s.k_size + s.v_size, reach or None, s.keep_first if reach or chunk else 0, chunk)
+                 if self.own_kv else None)
         if self._state_numbers() == 0:
             return paged
         if paged is None:
@@ -147,11 +150,15 @@ class WindowAttention:
         return PagedStateNeed(paged, StateNeed((self._state_numbers(),), torch.float32))
 
     def forward(self, x, step, cache):
+        ops = self.rt.ops
+        return ops.linear(self.inner(ops.linear(x, self.w_in), step, cache), self.w_o)
+
+    def inner(self, proj, step, cache, out=None, scale=1.0):
+        """From the rows ``[T, q | k | v | gate]`` to what the output product reads."""
         s, ops = self.spec, self.rt.ops
         if cache.writable != self.own_kv:
             raise ValueError("window attention: the schedule entry's cache does not fit the mixer "
                              "(a mixer without keys and values reads another entry's cache, and only such a mixer)")
-        proj = ops.linear(x, self.w_in)                      # [T, q | k | v | gate]
         gate = proj[:, self.channels:] if s.head_gate else None
         src = proj
         if self.w_conv is not None:
@@ -169,7 +176,6 @@ class WindowAttention:
                                   interleaved=getattr(self.position, "interleaved", False), positions=step.positions,
                                   slot_mapping=cache.slot_mapping, cache=cache.kv, values_from_keys=s.values_from_keys,
                                   **geometry, **rotation)
-        attn = ops.window_attention(q, cache=cache.kv, block_table=cache.block_table, step=step, scale=s.scale,
+        return ops.window_attention(q, cache=cache.kv, block_table=cache.block_table, step=step, scale=s.scale,
                                     window=s.window, keep_first=s.keep_first, softcap=s.softcap or 0.0, bias=self.bias,
-                                    sink=self.sink, gate=gate, **geometry)
-        return ops.linear(attn, self.w_o)
+                                    sink=self.sink, gate=gate, chunk=s.chunk, scale_out=scale, out=out, **geometry)

@@ -28,8 +28,8 @@ class FakeOps:
             self.clear_errors()
             raise RuntimeError(f"a kernel reported error code {code}")
 
-    def embedding(self, table, ids, out_dtype=None):
-        return table[ids.long()].to(out_dtype or table.dtype).clone()
+    def embedding(self, table, ids, out_dtype=None, scale=1.0):
+        return (table[ids.long()].to(out_dtype or table.dtype) * scale).clone()
 
     def rmsnorm(self, x, weight, eps, delta=None, rows=None):
         if rows is not None:
@@ -156,16 +156,21 @@ class FakeOps:
         return torch.tensor(out, dtype=torch.int32)
 
     # -- a 32-bit residual stream, mixers with state, attention over a latent, routed experts ---------------------
-    def rmsnorm_stream(self, h, weight, eps, delta=None, rows=None, out_dtype=torch.bfloat16):
+    def rmsnorm_stream(self, h, weight, eps, delta=None, rows=None, out_dtype=torch.bfloat16, scale=1.0, bias=None,
+                       again=None, vector=None):
         assert h.dtype == torch.float32
+        v = h.clone()
+        if delta is not None:
+            v = v + scale * (delta.float() + (bias if bias is not None else 0.0))
+        if again is not None:
+            table, ids, factor = again
+            v = v + factor * table[ids.long()].float()
+        if vector is not None:
+            v = v + vector
         if rows is not None:
-            v = h[rows.long()]
-            if delta is not None:
-                v = v + delta[rows.long()].float()
+            v = v[rows.long()]
         else:
-            if delta is not None:
-                h += delta.float()
-            v = h
+            h.copy_(v)
         return (v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * weight).to(out_dtype)
 
     def linear_batched(self, x, w, out_dtype=None, rotate=None, gate=None):
@@ -202,7 +207,7 @@ class FakeOps:
             hist.copy_(seq[seq.shape[0] - (taps - 1):])
         return out
 
-    def gated_delta_rule(self, qkv, ba, *, decay_log, decay_bias, state, step, heads, kv_heads, key_dim, value_dim,
+    def gated_delta_rule(self, qkv, beta, decay, *, decay_log, decay_bias, state, step, heads, kv_heads, key_dim, value_dim,
                          unit_eps, q_scale):
         T = qkv.shape[0]
         QK = kv_heads * key_dim
@@ -211,8 +216,9 @@ class FakeOps:
         v = qkv[:, 2 * QK:].float().view(T, heads, value_dim)
         q = q / torch.sqrt((q * q).sum(-1, keepdim=True) + unit_eps) * q_scale
         k = k / torch.sqrt((k * k).sum(-1, keepdim=True) + unit_eps)
-        beta = torch.sigmoid(ba[:, :heads].float())
-        decay = torch.exp(-torch.exp(decay_log) * torch.nn.functional.softplus(ba[:, heads:].float() + decay_bias))
+        beta = torch.sigmoid(beta.float())
+        a = torch.nn.functional.softplus(decay.float() + decay_bias).view(T, heads, -1)      # [.., 1] or [.., key_dim]
+        decay = torch.exp(-torch.exp(decay_log)[None, :, None] * a)
         out = torch.zeros(T, heads, value_dim)
         per = heads // kv_heads
         for lo, hi, slot in self._requests(step):
@@ -220,17 +226,37 @@ class FakeOps:
             for t in range(lo, hi):
                 for h in range(heads):
                     kk, qq = k[t, h // per], q[t, h // per]
-                    S[h] *= decay[t, h]
+                    S[h] *= decay[t, h][:, None]
                     u = beta[t, h] * (v[t, h] - S[h].T @ kk)
                     S[h] += torch.outer(kk, u)
                     out[t, h] = S[h].T @ qq
         return out
 
-    def gated_rmsnorm(self, o, gate, weight, eps):
+    def gated_rmsnorm(self, o, gate, weight, eps, activation="silu", scale=1.0, out=None):
         T, heads, vdim = o.shape
         g = gate.float().view(T, heads, vdim)
-        y = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * weight * (g * torch.sigmoid(g))
-        return y.reshape(T, heads * vdim).to(gate.dtype)
+        act = g * torch.sigmoid(g) if activation == "silu" else torch.sigmoid(g)
+        y = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * weight * act * scale
+        y = y.reshape(T, heads * vdim)
+        if out is None:
+            return y.to(gate.dtype)
+        return out.copy_(y)
+
+    def selective_scan(self, u, dt, bc, z, *, dt_bias, A, D, state, step, scale=1.0, out=None):
+        T, inner = u.shape
+        n = A.shape[1]
+        x, zz = u.float(), z.float()
+        dt = torch.nn.functional.softplus(dt + dt_bias)
+        B, C = bc[:, :n].float(), bc[:, n:2 * n].float()
+        if out is None:
+            out = torch.zeros(T, inner, dtype=u.dtype)
+        for lo, hi, slot in self._requests(step):
+            S = state[slot, :inner * n].view(inner, n)
+            for t in range(lo, hi):
+                S.copy_(torch.exp(dt[t][:, None] * A) * S + (dt[t] * x[t])[:, None] * B[t][None, :])
+                y = S @ C[t] + D * x[t]
+                out[t] = (y * zz[t] * torch.sigmoid(zz[t]) * scale).to(u.dtype)
+        return out
 
     def rglru_scan(self, u, gates, y_pre, *, y_bias, r_bias, i_bias, lam, decay_scale, state, step, blocks):
         T, W = u.shape
@@ -531,19 +557,24 @@ class FakeOps:
         return q
 
     def window_attention(self, q, *, cache, block_table, step, scale, window, keep_first, softcap, bias, sink, gate, heads,
-                         kv_heads, key_dim, value_dim):
+                         kv_heads, key_dim, value_dim, chunk=0, scale_out=1.0, out=None):
         T = q.shape[0]
         page_size = cache.shape[1]
         nk = kv_heads * key_dim
-        out = torch.zeros(T, heads, value_dim)
+        into, out = out, torch.zeros(T, heads, value_dim)
         for t in range(T):
             r = int(step.request_of_row[t])
             if r < 0:
                 continue
             p = int(step.positions[t])
             js = torch.arange(0, p + 1)
-            if window:
-                js = js[(p - js < window) | (js < keep_first)]
+            if window or chunk:
+                seen = torch.ones_like(js, dtype=torch.bool)
+                if window:
+                    seen &= p - js < window
+                if chunk:
+                    seen &= js // chunk == p // chunk
+                js = js[seen | (js < keep_first)]
             pages = block_table[r, (js // page_size).long()].long()
             if not (pages >= 0).all():
                 self._report(2)
@@ -565,8 +596,9 @@ class FakeOps:
                 o = (e / den) @ V[:, g]
                 if gate is not None:
                     o = o * torch.sigmoid(gate[t, h].float())
-                out[t, h] = o
-        return out.reshape(T, heads * value_dim).to(q.dtype)
+                out[t, h] = o * scale_out
+        out = out.reshape(T, heads * value_dim).to(q.dtype)
+        return out if into is None else into.copy_(out)
 
     # -- a bigram embedding, rotations by computed angles, gates a column, two-matrix experts -----------------------------
     def embed_bigram(self, table, bigram, step, *, state, mul_prev, mul_cur, buckets, out_dtype=None):
@@ -598,9 +630,15 @@ class FakeOps:
         g = gate.float()
         return (a.float() * (torch.sigmoid(g) if kind == "sigmoid" else g * torch.sigmoid(g))).to(a.dtype)
 
-    def activation(self, z, kind):
+    def activation(self, z, kind, bias=None):
+        v = z.float() + (bias if bias is not None else 0.0)
+        if kind == "gelu_erf":
+            return (0.5 * v * (1.0 + torch.erf(v * 0.5 ** 0.5))).to(z.dtype)
         assert kind == "relu2"
-        return (torch.relu(z.float()) ** 2).to(z.dtype)
+        return (torch.relu(v) ** 2).to(z.dtype)
+
+    def linear_bias_gelu(self, x, w, bias):
+        return self.activation(self.linear(x, w), "gelu_erf", bias)
 
     def scale_(self, x, scale):
         return x.mul_(scale)

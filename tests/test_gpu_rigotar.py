@@ -331,8 +331,8 @@ def test_delta_rule_recalls_a_value_written_long_ago():
     outs, at = [], 0
     for cut in (7, 100, 1, 1, 2, 109):                                           # the state is carried over these steps
         step = _step([0] * cut, [0] * cut, [0, 0, cut], [-1, 1])                  # (a request of padding in front)
-        outs.append(ops.gated_delta_rule(qkv[at:at + cut], ba[at:at + cut], decay_log=zeros, decay_bias=zeros, state=state,
-                                         step=step, heads=heads, kv_heads=kv_heads, key_dim=D, value_dim=V,
+        outs.append(ops.gated_delta_rule(qkv[at:at + cut], ba[at:at + cut, :heads], ba[at:at + cut, heads:], decay_log=zeros,
+                                         decay_bias=zeros, state=state, step=step, heads=heads, kv_heads=kv_heads, key_dim=D, value_dim=V,
                                          unit_eps=1e-6, q_scale=1.0))
         at += cut
     ops.check_errors()
@@ -369,9 +369,9 @@ def test_delta_rule_kernels_of_every_key_size(dim, vdim, dtype):
     rows1 = list(range(20)) + list(range(lens[0], T))
     rows2 = list(range(20, lens[0]))
     sel1, sel2 = torch.tensor(rows1), torch.tensor(rows2)
-    out1 = ops.gated_delta_rule(qkv[sel1].to(DEV).contiguous(), ba[sel1].to(DEV).contiguous(),
+    out1 = ops.gated_delta_rule(qkv[sel1].to(DEV).contiguous(), ba[sel1, :heads].to(DEV), ba[sel1, heads:].to(DEV),
                                 step=_step([0] * len(rows1), [0] * len(rows1), [0, 20, len(rows1)], [2, 0]), **kw)
-    out2 = ops.gated_delta_rule(qkv[sel2].to(DEV).contiguous(), ba[sel2].to(DEV).contiguous(),
+    out2 = ops.gated_delta_rule(qkv[sel2].to(DEV).contiguous(), ba[sel2, :heads].to(DEV), ba[sel2, heads:].to(DEV),
                                 step=_step([0] * len(rows2), [0] * len(rows2), [0, len(rows2)], [2]), **kw)
     ops.check_errors()
     got = torch.zeros(T, heads, vdim, dtype=F64)
