@@ -392,6 +392,29 @@ def _sagelorn_config(width: int, layers: int, kinds=("attention", "latent_attent
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}, "layers": out}
 
 
+def _kedavik_config(width: int, layers: int, kinds=("mamba1", "parallel"), mlp: bool = True, chunk: int = 1024, loop=None,
+                    vocab: int = 32768):
+    """Layer sizes that resemble a real model's at this width: a scan over twice the width with 16 states a channel and
+    step sizes through a sixteenth of the width; beside each other half as many 128-wide attention heads as the dense
+    decoder's (half as many key/value heads, whole heads rotated, chunks of ``chunk`` places) and as many 128 x 128 delta
+    heads as Rigotar's, decays and gate through 128 numbers; a two-matrix feed-forward of four times the width behind the
+    pair."""
+    heads = width // 128
+    mixers = {"mamba1": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4},
+              "parallel": {"left": {"heads": heads, "kv_heads": max(1, heads // 2), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                    "rot": {"dims": 128, "base": 1e6}, "mask": {"size": chunk}},
+                           "right": {"heads": heads, "kv_heads": max(1, heads // 2), "dim": 128, "vdim": 128, "conv": 4,
+                                     "decay_rank": 128, "gate_rank": 128}, "left_scale": 0.8, "right_scale": 0.6}}
+    out = {"architecture": "Kedavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 0.5},
+           "residual_mult": 0.4,
+           "layers": [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]],
+                       "mlp": {"kind": "dense", "ff": 4 * width} if mlp and kinds[i % len(kinds)] == "parallel" else None}
+                      for i in range(layers)]}
+    if loop is not None:
+        out["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return out
+
+
 def _dense_config(width: int, layers: int, vocab: int = 32768):
     return dict(QWEN3_0_6B, hidden_size=width, intermediate_size=3 * width, num_hidden_layers=layers,
                 num_attention_heads=width // 128 * 2, num_key_value_heads=width // 128, head_dim=128, vocab_size=vocab,
@@ -453,6 +476,129 @@ def _timed_steps(model, batch: int, context: int, prompt: int, steps: int):
     return sorted(pre[2:])[len(pre[2:]) // 2], dec
 
 
+def _graph_us(fn, sets, calls: int = 24, repeats: int = 5) -> float:
+    """Microseconds of one call as a step sees it: ``calls`` calls in a row on ``sets`` different inputs inside one CUDA
+    graph, device-timed, median of ``repeats`` replays."""
+    import torch
+    for i in range(sets):
+        fn(i)
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for c in range(calls):
+            fn(c % sets)
+    graph.replay()
+    times = []
+    for _ in range(repeats):
+        torch.cuda.synchronize()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        graph.replay()
+        b.record()
+        torch.cuda.synchronize()
+        times.append(a.elapsed_time(b) / calls * 1e3)
+    return sorted(times)[len(times) // 2]
+
+
+def _kedavik_kernels(width: int, batch: int, prompt: int, context: int):
+    """The kernels of the Kedavik design beside the like kernel of another design, one prompt of ``prompt`` tokens and one
+    decode step of ``batch`` requests: microseconds a call, the bytes that it has to move, and the fraction of the
+    measured copy bandwidth that this makes.  Several sets of inputs and states in turn, together larger than L2."""
+    import types
+    import torch
+    from pih_b200.kernels import get_ops
+    ops = get_ops(torch.device("cuda:0"))
+    hbm = peaks()[0]
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    heads, d, n, inner, group = width // 128, 128, 16, 2 * width, 2
+    rows_out = []
+
+    def steps_of(decode):
+        counts = [1] * batch if decode else [prompt]
+        starts = [context - 1] * batch if decode else [0]
+        cu = [0]
+        for c in counts:
+            cu.append(cu[-1] + c)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        return types.SimpleNamespace(
+            num_requests=len(counts), cu_q=i32(cu), q_start=i32(starts), state_slots=i32(range(len(counts))),
+            host_cu_q=cu, host_q_start=starts, attention_plans={}, meta=None,
+            request_of_row=i32([r for r, c in enumerate(counts) for _ in range(c)]),
+            positions=i32([starts[r] + i for r, c in enumerate(counts) for i in range(c)])), cu[-1], len(counts)
+
+    for decode in (False, True):
+        step, T, R = steps_of(decode)
+        sets = 24 if decode else 6
+        rnd = lambda *shape, dtype=bf: [torch.randn(*shape, device=dev, dtype=dtype) for _ in range(sets)]
+
+        def add(name, us, nbytes):
+            rows_out.append({"kernel": name, "width": width, "step": f"decode x{batch}" if decode else f"prompt {prompt}",
+                             "us": round(us, 2), "MB": round(nbytes / 1e6, 2),
+                             "of_copy_peak": round(nbytes / (us * 1e-6) / (hbm * 1e9), 4)})
+
+        # the scan beside the other diagonal recurrence (both with what makes their coefficients)
+        u, dt, bc, z = rnd(T, inner), rnd(T, inner, dtype=f32), rnd(T, 2 * n), rnd(T, inner)
+        st = rnd(R, inner * n, dtype=f32)
+        A, vec = -torch.rand(inner, n, device=dev), torch.randn(inner, device=dev)
+        add("selective_scan", _graph_us(lambda i: ops.selective_scan(u[i], dt[i], bc[i], z[i], dt_bias=vec, A=A, D=vec, state=st[i],
+                                                                     step=step), sets),
+            T * (inner * (2 + 4 + 2 + 2) + 4 * n) + (2 * R + 1) * inner * n * 4)
+        del u, dt, bc, z, st
+        W = width
+        u, gates, y, st = rnd(T, W), rnd(T, heads, 2 * W // heads, dtype=f32), rnd(T, W), rnd(R, W, dtype=f32)
+        v = torch.randn(W, device=dev)
+        add("rglru_scan (Rigotar)", _graph_us(lambda i: ops.rglru_scan(u[i], gates[i], y[i], y_bias=v, r_bias=v, i_bias=v, lam=v,
+                                                                       decay_scale=8.0, state=st[i], step=step, blocks=heads), sets),
+            T * W * (2 + 8 + 2 + 2) + 2 * R * W * 4)
+        del u, gates, y, st
+        # the delta rule with a decay a key channel beside the one with a decay a head
+        G = max(1, heads // group)
+        qkv, b, st = rnd(T, (2 * G + heads) * d), rnd(T, heads), rnd(R, heads * d * d, dtype=f32)
+        log, fixed = torch.zeros(heads, device=dev), T * ((2 * G + heads) * d * 2 + heads * 2 + heads * d * 4) + 2 * R * heads * d * d * 4
+        kw = dict(decay_log=log, step=step, heads=heads, kv_heads=G, key_dim=d, value_dim=d, unit_eps=1e-6, q_scale=d ** -0.5)
+        a, bias = rnd(T, heads * d, dtype=f32), torch.randn(heads * d, device=dev)
+        add("gated_delta_rule, decay a channel",
+            _graph_us(lambda i: ops.gated_delta_rule(qkv[i], b[i], a[i], decay_bias=bias, state=st[i], **kw), sets),
+            fixed + T * heads * d * 4)
+        a, bias = rnd(T, heads), torch.randn(heads, device=dev)
+        add("gated_delta_rule, decay a head (Rigotar)",
+            _graph_us(lambda i: ops.gated_delta_rule(qkv[i], b[i], a[i], decay_bias=bias, state=st[i], **kw), sets),
+            fixed + T * heads * 2)
+        del qkv, b, st, a
+        # attention inside chunks beside the same attention over a window of as many keys
+        pages = -(-context // PAGE)
+        tables = torch.arange(R * pages, dtype=torch.int32, device=dev).view(R, pages)
+        q, cache, gate = rnd(T, heads * d), rnd(R * pages, PAGE, 2 * G * d), rnd(T, heads)
+        sink = torch.zeros(heads, device=dev)
+        span = 1024
+        common = dict(block_table=tables, step=step, scale=d ** -0.5, keep_first=0, softcap=0.0, bias=None, heads=heads,
+                      kv_heads=G, key_dim=d, value_dim=d)
+        seen = R * span if decode else prompt
+        nbytes = T * heads * d * 4 + seen * 2 * G * d * 2
+        add(f"window_attention, chunks of {span}, gate a head",
+            _graph_us(lambda i: ops.window_attention(q[i], cache=cache[i], window=0, chunk=span, sink=None, gate=gate[i], **common), sets),
+            nbytes)
+        add(f"window_attention, window of {span}, sink (Sagelorn)",
+            _graph_us(lambda i: ops.window_attention(q[i], cache=cache[i], window=span, sink=sink, gate=None, **common), sets),
+            nbytes)
+        del q, cache, gate
+        # the norm of the stream with everything that a pass of the loop adds, beside the plain one; the two activations
+        h, y = rnd(T, width, dtype=f32), rnd(T, width)
+        table, ids = torch.randn(32768, width, device=dev, dtype=bf), torch.randint(0, 32768, (T,), dtype=torch.int32, device=dev)
+        wv = torch.randn(width, device=dev)
+        add("rmsnorm_stream, factor, bias, embedding, vector",
+            _graph_us(lambda i: ops.rmsnorm_stream(h[i], wv, 1e-6, delta=y[i], scale=0.4, bias=wv, again=(table, ids, 0.5), vector=wv), sets),
+            T * width * (8 + 2 + 2 + 2))
+        add("rmsnorm_stream (Rigotar)", _graph_us(lambda i: ops.rmsnorm_stream(h[i], wv, 1e-6, delta=y[i]), sets), T * width * (8 + 2 + 2))
+        zz, bz = rnd(T, 4 * width), torch.randn(4 * width, device=dev)
+        add("activation gelu_erf with bias", _graph_us(lambda i: ops.activation(zz[i], "gelu_erf", bz), sets), T * 16 * width)
+        add("bias_xielu (Tuganex)", _graph_us(lambda i: ops.bias_xielu(zz[i], bz, 0.8, 0.8), sets), T * 16 * width)
+        del h, y, zz
+        torch.cuda.empty_cache()
+    ops.check_errors()
+    return rows_out
+
+
 def design_run(args) -> int:
     """``--design rigotar``: prompt and decode throughput of the Rigotar design at two widths with layer sizes that
     resemble a real model's (random weights, bf16), beside the dense decoder at the same width, depth and number of
@@ -463,7 +609,24 @@ def design_run(args) -> int:
     batch, context, prompt, steps = args.batch, CONTEXT, PREFILL_TOKENS, max(8, args.steps // 4)
     with ClockSampler() as clocks:
         for width in (1024, 2048):
-            if args.design == "sagelorn":
+            if args.design == "kedavik":
+                # the design beside the model nearest to it (a diagonal recurrence, a delta rule, attention) and the dense
+                # decoder; and each of its kinds of layer alone beside its like
+                cases = [("kedavik", _kedavik_config(width, 8)), ("rigotar", _rigotar_config(width, 8)),
+                         ("dense", _dense_config(width, 8))]
+                if width == 1024:
+                    cases += [(f"kedavik {k} x4, no feed-forward", _kedavik_config(width, 4, kinds=(k,), mlp=False))
+                              for k in ("mamba1", "parallel")]
+                    cases += [("rigotar rglru x4, no feed-forward", _rigotar_config(width, 4, kinds=("rglru",), moe=False)),
+                              ("rigotar delta x4, no feed-forward", _rigotar_config(width, 4, kinds=("delta",), moe=False)),
+                              ("sagelorn attention x4, no feed-forward",
+                               _sagelorn_config(width, 4, kinds=("attention",), mlps=None, share=False)),
+                              ("kedavik parallel x4, dense feed-forward", _kedavik_config(width, 4, kinds=("parallel",))),
+                              ("tuganex retention x4, no feed-forward", _tuganex_config(width, 4, kinds=("retention",), mlps=None)),
+                              ("tuganex retention x4, dense feed-forward",
+                               _tuganex_config(width, 4, kinds=("retention",), mlps=("dense",))),
+                              ("kedavik 2 layers run 4 times", _kedavik_config(width, 4, loop=(1, 3, 4)))]
+            elif args.design == "sagelorn":
                 # the design beside the model nearest to it (norms on the outputs, retention, shared caches, routed experts
                 # with a shared one) and the dense decoder; and each of its kinds of layer alone beside its like
                 cases = [("sagelorn", _sagelorn_config(width, 8)), ("tuganex", _tuganex_config(width, 8, share_from=6)),
@@ -521,12 +684,13 @@ def design_run(args) -> int:
                 del model
                 gc.collect()
                 torch.cuda.empty_cache()
+        kernels = {"kernels": _kedavik_kernels(1024, batch, prompt, context)} if args.design == "kedavik" else {}
         clock_summary = clocks.summary()
     print(json.dumps({"metric": f"prompt and decode tok/s of the {args.design.capitalize()} design beside the framework's other models",
                       "dtype": "bf16",
                       "data": "synthetic", "n_gpus": 1, "config": {"prompt_tokens": prompt, "decode_batch": batch,
                                                                    "context": context, "page_size": PAGE},
-                      "rows": rows, "clocks": clock_summary}))
+                      "rows": rows, **kernels, "clocks": clock_summary}))
     return 0
 
 
@@ -549,7 +713,7 @@ def main() -> int:
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
-    ap.add_argument("--design", default=None, choices=["rigotar", "tuganex", "pegopel", "sagelorn"],
+    ap.add_argument("--design", default=None, choices=["rigotar", "tuganex", "pegopel", "sagelorn", "kedavik"],
                     help="instead of the recorded workload: this design's prompt and decode throughput beside the dense decoder's")
     ap.add_argument("--plain-launches", action="store_true",
                     help="launch kernels fully serialised instead of with programmatic dependent launch")

@@ -81,10 +81,14 @@ selective_scan_kernel(const ScanArgs p) {
   constexpr int NP = kParts * kN;                                       // states with the padding
   constexpr int E = (kScanRows * CH + TH - 1) / TH;                     // (row, channel) pairs a thread
   constexpr int EB = kScanRows * 2 * NP / TH;                           // numbers of B and C a thread
-  static_assert(kScanRows * 2 * NP % TH == 0, "whole shares");
-  __shared__ __align__(16) float2 steps[kScanRows][CH];                 // (dt, dt x)
-  __shared__ __align__(16) float bc_s[kScanRows][2][NP];
-  __shared__ float y_s[kScanRows][CH];
+  static_assert(kScanRows * 2 * NP % TH == 0 && kN % 2 == 0, "whole shares, 8-byte loads");
+  extern __shared__ __align__(16) float scan_smem[];
+  typedef float2 (*Steps)[CH];
+  typedef float (*Vectors)[2][NP];
+  typedef float (*Outputs)[CH];
+  Vectors bc_s = reinterpret_cast<Vectors>(scan_smem);                  // [rows][B, C][NP]
+  Steps steps = reinterpret_cast<Steps>(scan_smem + kScanRows * 2 * NP);                    // [rows][CH]: (dt, dt x)
+  Outputs y_s = reinterpret_cast<Outputs>(scan_smem + kScanRows * (2 * NP + 2 * CH));       // [rows][CH]
   wait_for_prior_kernels();
   launch_dependents();
   const int r = blockIdx.x, c0 = blockIdx.y * CH, tid = threadIdx.x;
@@ -112,63 +116,70 @@ selective_scan_kernel(const ScanArgs p) {
     bias[e] = ce < p.inner ? p.dt_bias[ce] : 0.0f;
     skip[e] = ce < p.inner ? p.D[ce] : 0.0f;
   }
-  float nx[E], nz[E], nt[E], nbc[EB];                                   // the next chunk's numbers
+  // the next chunk's numbers, as they lie in memory: nothing is computed from them before they are needed
+  T nx[E], nz[E], nbc[EB];
+  float nt[E];
+  const T zero = from_float<T>(0.0f);
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int e = 0; e < E; ++e) {
       const int idx = tid + e * TH, t = t0 + idx / CH, ce = c0 + idx % CH;
       const bool there = idx < kScanRows * CH && t < hi && ce < p.inner;
-      nx[e] = there ? to_float<T>(u[t * p.ldu + ce]) : 0.0f;
-      nz[e] = there ? to_float<T>(z[t * p.ldz + ce]) : 0.0f;
+      nx[e] = there ? u[t * p.ldu + ce] : zero;
+      nz[e] = there ? z[t * p.ldz + ce] : zero;
       nt[e] = there ? p.dt[t * p.lddt + ce] : 0.0f;
     }
 #pragma unroll
     for (int e = 0; e < EB; ++e) {
       const int idx = tid + e * TH, t = t0 + idx / (2 * NP), which = (idx / NP) & 1, n = idx % NP;
-      nbc[e] = t < hi && n < p.states ? to_float<T>(bc[t * p.ldbc + which * p.states + n]) : 0.0f;
+      nbc[e] = t < hi && n < p.states ? bc[t * p.ldbc + which * p.states + n] : zero;
     }
   };
   fetch(lo);
   for (int t0 = lo; t0 < hi; t0 += kScanRows) {
     const int n_rows = min(kScanRows, hi - t0);
-    float x[E], zz[E];
+    float x[E];
+    T zz[E];
 #pragma unroll
     for (int e = 0; e < E; ++e) {
       const int idx = tid + e * TH;
-      x[e] = nx[e];
+      x[e] = to_float<T>(nx[e]);
       zz[e] = nz[e];
       const float dt = softplus_f(nt[e] + bias[e]);
-      if (idx < kScanRows * CH) steps[idx / CH][idx % CH] = make_float2(dt, dt * nx[e]);
+      if (idx < kScanRows * CH) steps[idx / CH][idx % CH] = make_float2(dt, dt * x[e]);
     }
 #pragma unroll
-    for (int e = 0; e < EB; ++e) (&bc_s[0][0][0])[tid + e * TH] = nbc[e];
+    for (int e = 0; e < EB; ++e) scan_smem[tid + e * TH] = to_float<T>(nbc[e]);
     __syncthreads();
     if (t0 + kScanRows < hi) fetch(t0 + kScanRows);
     float share[kScanRows];
+    auto row = [&](int t) {
+      const float2 st = steps[t][cl];
+      float B[kN], C[kN];
 #pragma unroll
-    for (int t = 0; t < kScanRows; ++t) {
-      share[t] = 0.0f;
-      if (t < n_rows) {                                                 // (the same for the whole block)
-        const float2 st = steps[t][cl];
-        float B[kN], C[kN];
-        if constexpr (kN % 4 == 0) {
+      for (int i = 0; i < kN; i += 2) {
+        const float2 b2 = *reinterpret_cast<const float2*>(&bc_s[t][0][n0 + i]);
+        const float2 c2 = *reinterpret_cast<const float2*>(&bc_s[t][1][n0 + i]);
+        B[i] = b2.x; B[i + 1] = b2.y;
+        C[i] = c2.x; C[i + 1] = c2.y;
+      }
+      float y = 0.0f;
 #pragma unroll
-          for (int i = 0; i < kN; i += 4) {
-            const float4 b4 = *reinterpret_cast<const float4*>(&bc_s[t][0][n0 + i]);
-            const float4 c4 = *reinterpret_cast<const float4*>(&bc_s[t][1][n0 + i]);
-            B[i] = b4.x; B[i + 1] = b4.y; B[i + 2] = b4.z; B[i + 3] = b4.w;
-            C[i] = c4.x; C[i + 1] = c4.y; C[i + 2] = c4.z; C[i + 3] = c4.w;
-          }
-        } else {
+      for (int i = 0; i < kN; ++i) {
+        if (kExact) S[i] = fmaf(expm1f(st.x * A[i]), S[i], fmaf(st.y, B[i], S[i]));
+        else S[i] = fmaf(mma::exp2_fast(st.x * A[i]), S[i], st.y * B[i]);
+        y = fmaf(S[i], C[i], y);
+      }
+      share[t] = y;
+    };
+    if (n_rows == kScanRows) {                                          // (the same for the whole block; no branch a row, so
+#pragma unroll                                                          // that the rows' loads and exponentials overlap)
+      for (int t = 0; t < kScanRows; ++t) row(t);
+    } else {
 #pragma unroll
-          for (int i = 0; i < kN; ++i) { B[i] = bc_s[t][0][n0 + i]; C[i] = bc_s[t][1][n0 + i]; }
-        }
-#pragma unroll
-        for (int i = 0; i < kN; ++i) {
-          if (kExact) S[i] = fmaf(expm1f(st.x * A[i]), S[i], fmaf(st.y, B[i], S[i]));
-          else S[i] = fmaf(mma::exp2_fast(st.x * A[i]), S[i], st.y * B[i]);
-          share[t] = fmaf(S[i], C[i], share[t]);
-        }
+      for (int t = 0; t < kScanRows; ++t) {
+        share[t] = 0.0f;
+        if (t < n_rows) row(t);
       }
     }
     const int first = fold_shares<kScanRows, kParts / 2>(share, part);
@@ -181,7 +192,7 @@ selective_scan_kernel(const ScanArgs p) {
       const int idx = tid + e * TH, t = idx / CH, ce = c0 + idx % CH;
       if (idx < kScanRows * CH && t < n_rows && ce < p.inner) {
         const float y = fmaf(skip[e], x[e], y_s[t][idx % CH]);
-        out[(t0 + t) * p.ldo + ce] = from_float<T>(silu_times<T>(zz[e], y) * p.out_scale);
+        out[(t0 + t) * p.ldo + ce] = from_float<T>(silu_times<T>(to_float<T>(zz[e]), y) * p.out_scale);
       }
     }
     // (y_s is written again only behind the next chunk's first barrier, steps and bc_s only behind this chunk's second)
@@ -196,18 +207,28 @@ selective_scan_kernel(const ScanArgs p) {
 template <typename T, int kParts, int kN>
 static void launch_scan(const ScanArgs& p, int requests, cudaStream_t s) {
   constexpr int CH = ScanShape<kParts>::CH;
-  launch_kernel(selective_scan_kernel<T, kParts, kN>, dim3(requests, (p.inner + CH - 1) / CH),
-                dim3(ScanShape<kParts>::kThreads), 0, s, p);
+  const dim3 grid(requests, (p.inner + CH - 1) / CH);
+  const int needed = kScanRows * (2 * kParts * kN + 3 * CH) * static_cast<int>(sizeof(float));
+  // the rows follow one another: with no more blocks than SMs every block asks for more than half of an SM's shared memory
+  // and so gets an SM alone
+  const bool alone = static_cast<long long>(grid.x) * grid.y <= 148;
+  const int smem = alone && needed < 116 * 1024 ? 116 * 1024 : needed;
+  static int raised = 48 * 1024;                               // (per instance)
+  if (smem > raised) {
+    cudaFuncSetAttribute(selective_scan_kernel<T, kParts, kN>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    raised = smem;
+  }
+  launch_kernel(selective_scan_kernel<T, kParts, kN>, grid, dim3(ScanShape<kParts>::kThreads), smem, s, p);
 }
 
 template <typename T>
 static int dispatch_scan(const ScanArgs& p, int requests, cudaStream_t s) {
   const int n = p.states;
-  if (n <= 4) launch_scan<T, 1, 4>(p, requests, s);
-  else if (n <= 8) launch_scan<T, 2, 4>(p, requests, s);
-  else if (n <= 16) launch_scan<T, 4, 4>(p, requests, s);
-  else if (n <= 32) launch_scan<T, 8, 4>(p, requests, s);
-  else if (n <= 64) launch_scan<T, 16, 4>(p, requests, s);
+  if (n <= 4) launch_scan<T, 2, 2>(p, requests, s);
+  else if (n <= 8) launch_scan<T, 4, 2>(p, requests, s);
+  else if (n <= 16) launch_scan<T, 8, 2>(p, requests, s);
+  else if (n <= 32) launch_scan<T, 16, 2>(p, requests, s);
+  else if (n <= 64) launch_scan<T, 32, 2>(p, requests, s);
   else if (n <= 128) launch_scan<T, 32, 4>(p, requests, s);
   else if (n <= 256) launch_scan<T, 32, 8>(p, requests, s);
   else return PIH_ERR_UNSUPPORTED;

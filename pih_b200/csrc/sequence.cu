@@ -287,37 +287,58 @@ causal_conv_history_kernel(const T* __restrict__ x, long long ldx, const float* 
     if (j < hist_n) st[static_cast<long long>(j) * channels + c] = keep[j];
 }
 
-// One block a row.  qk: [rows, ld] with q heads at column 0 and k heads at column kv_heads*dim (after convolution and
+// Block (row, part): part 0 the vectors and the write strengths — and the decays, where it is the only part —, part p > 0 the
+// decays kDecaySlice (p - 1) and on.  qk: [rows, ld] with q heads at column 0 and k heads at column kv_heads*dim (after convolution and
 // activation); b: [rows, ldb] write-strength logits a head; a: [rows, lda] decay logits, one a head or (``channels``) one a
 // head and key channel, [heads, dim], with a bias of the same layout; decay_log: one a head.
-// qn, kn: fp32 [rows, kv_heads, dim]; decay (as g - 1): fp32 [rows, heads] or [rows, heads, dim]; beta: fp32 [rows, heads].
+// qn, kn: fp32 [rows, kv_heads, dim]; qk_dot: their product k . q, fp32 [rows, kv_heads]; decay (as g - 1): fp32 [rows,
+// heads] or [rows, heads, dim]; beta: fp32 [rows, heads].
+constexpr int kDecaySlice = 512;
+
 template <typename T, typename TA>
 __global__ void __launch_bounds__(128)
 delta_prepare_kernel(const T* __restrict__ qk, long long ld, const T* __restrict__ b, long long ldb,
                      const TA* __restrict__ a, long long lda, int channels,
                      const float* __restrict__ decay_log, const float* __restrict__ decay_bias, float* __restrict__ qn,
-                     float* __restrict__ kn, float* __restrict__ decay, float* __restrict__ beta, int heads, int kv_heads,
-                     int dim, float unit_eps, float q_scale) {
+                     float* __restrict__ kn, float* __restrict__ qk_dot, float* __restrict__ decay, float* __restrict__ beta,
+                     int heads, int kv_heads, int dim, float unit_eps, float q_scale) {
   wait_for_prior_kernels();
   launch_dependents();
   const int row = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-  for (int v = warp; v < 2 * kv_heads; v += warps) {             // vector v: q head v, or k head v - kv_heads
-    const T* src = qk + static_cast<long long>(row) * ld + static_cast<long long>(v) * dim;
-    float ss = 0.0f;
-    for (int i = lane; i < dim; i += 32) { const float a = to_float<T>(src[i]); ss = fmaf(a, a, ss); }
-    ss = warp_sum(ss);
-    const float scale = (1.0f / sqrtf(ss + unit_eps)) * (v < kv_heads ? q_scale : 1.0f);
-    float* dst = (v < kv_heads ? qn : kn) + (static_cast<long long>(row) * kv_heads + (v < kv_heads ? v : v - kv_heads)) * dim;
-    for (int i = lane; i < dim; i += 32) dst[i] = to_float<T>(src[i]) * scale;
+  for (int g = warp; g < kv_heads && blockIdx.y == 0; g += warps) {
+    const T* q = qk + static_cast<long long>(row) * ld + static_cast<long long>(g) * dim;
+    const T* k = q + static_cast<long long>(kv_heads) * dim;
+    float sq = 0.0f, sk = 0.0f;
+    for (int i = lane; i < dim; i += 32) {
+      const float x = to_float<T>(q[i]), y = to_float<T>(k[i]);
+      sq = fmaf(x, x, sq);
+      sk = fmaf(y, y, sk);
+    }
+    sq = (1.0f / sqrtf(warp_sum(sq) + unit_eps)) * q_scale;
+    sk = 1.0f / sqrtf(warp_sum(sk) + unit_eps);
+    const long long at = (static_cast<long long>(row) * kv_heads + g) * dim;
+    float dot = 0.0f;
+    for (int i = lane; i < dim; i += 32) {
+      const float x = to_float<T>(q[i]) * sq, y = to_float<T>(k[i]) * sk;
+      qn[at + i] = x;
+      kn[at + i] = y;
+      dot = fmaf(x, y, dot);
+    }
+    dot = warp_sum(dot);
+    if (lane == 0) qk_dot[static_cast<long long>(row) * kv_heads + g] = dot;
   }
-  for (int h = threadIdx.x; h < heads; h += blockDim.x) {
+  for (int h = threadIdx.x; h < heads && blockIdx.y == 0; h += blockDim.x) {
     beta[static_cast<long long>(row) * heads + h] = sigmoid_f(to_float<T>(b[static_cast<long long>(row) * ldb + h]));
   }
   // g - 1 rather than g: a decay next to 1 keeps its distance from 1 to full precision (see rglru_gates_kernel)
   const int per = channels ? dim : 1;
   const long long row_a = static_cast<long long>(row) * lda, row_g = static_cast<long long>(row) * heads * per;
-  for (int i = threadIdx.x; i < heads * per; i += blockDim.x)
+  const bool sliced = gridDim.y > 1;
+  if (sliced && blockIdx.y == 0) return;
+  const int from = sliced ? (static_cast<int>(blockIdx.y) - 1) * kDecaySlice : 0;
+  const int to = sliced ? min(heads * per, from + kDecaySlice) : heads * per;
+  for (int i = from + threadIdx.x; i < to; i += blockDim.x)
     decay[row_g + i] = expm1f(-expf(decay_log[i / per]) * softplus_f(to_float<TA>(a[row_a + i]) + decay_bias[i]));
 }
 
@@ -412,13 +433,31 @@ __global__ void delta_recurrence_kernel(const float* __restrict__ qn, const floa
     for (int i = 0; i < dim; ++i) Sg[static_cast<long long>(i) * vdim + col] = S[i * cols + j];
 }
 
-// The same recurrence with S in registers, for the key sizes that have an instance.  Block (request, head, 32 value
-// columns); a column of S is held by 8 threads (4 for small keys), thread (column c = tid / parts, part p = tid % parts)
-// the rows p * kDim / parts ..., so the parts of a column sit in neighbouring lanes and meet through shuffles.  What the recurrence reads of a
-// token (k, q, the block's 32 values, decay, write strength) is staged in shared memory a chunk of tokens at a time,
-// two buffers: the next chunk's numbers are copied asynchronously while this chunk is computed, so no load from
-// memory and only one barrier a chunk lie on the chain from token to token.  The order of the
-// additions is fixed by the kernel, not by the step's make-up or by where a chunk begins.
+// The same recurrence with S in registers, for the key sizes that have an instance.  Block (request, head, 16 value
+// columns); a column of S is held by 8 threads (4 for small keys, 16 for 256), thread (column c = tid / parts, part p = tid %
+// parts) every parts-th piece of four rows from piece p on: the parts of a column sit in neighbouring lanes, meet through
+// shuffles, and read neighbouring 16-byte pieces of k and q (no bank conflicts).
+//
+// What a token costs is the chain from its state to the next one's, so both products that read the state are taken from the
+// SAME (decayed) state g S and meet in the same shuffles: with a = (g S)^T k and b = (g S)^T q,
+//     u = beta (v - a),    o = b + (k . q) u,    S <- g S + k u^T
+// — the read-out of the state after the write, without reading it again; k . q comes from delta_prepare.  Products and
+// updates take two numbers an instruction (fma.rn.f32x2: each half rounds as fma.rn.f32 does).
+//
+// What the recurrence reads of a token (k, q, k . q, the block's values, decay, write strength) is staged in shared memory
+// a chunk of tokens at a time, two buffers: the next chunk's numbers are copied asynchronously while this chunk is computed,
+// so no load from memory and only one barrier a chunk lie on the chain from token to token; a token's numbers go from there
+// to registers one token ahead.  The order of the additions is fixed by the kernel, not by the step's make-up or by where a
+// chunk begins.  With kChannel the decay (as g - 1, [rows, heads, kDim]) multiplies the rows of S; it is staged like k and q.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("{\n\t.reg .b64 ra, rb, rc, rd;\n\t"
+      "mov.b64 ra, {%2, %3};\n\tmov.b64 rb, {%4, %5};\n\tmov.b64 rc, {%6, %7};\n\t"
+      "fma.rn.f32x2 rd, ra, rb, rc;\n\tmov.b64 {%0, %1}, rd;\n\t}"
+      : "=f"(d.x), "=f"(d.y)
+      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+  return d;
+}
 __device__ __forceinline__ void async_copy_16(void* smem_dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst))), "l"(src));
 }
@@ -428,122 +467,129 @@ __device__ __forceinline__ void async_copy_4(void* smem_dst, const void* src) {
 __device__ __forceinline__ void async_copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void async_copies_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// With kChannel the decay (as g - 1, [rows, heads, kDim]) multiplies the rows of S; it is staged like k and q.
 template <int kDim, bool kChannel>
 struct DeltaShape {
-  static constexpr int kParts = kDim >= 256 && kChannel ? 16 : (kDim >= 64 ? 8 : 4);   // threads a column of S
-  static constexpr int kThreads = 32 * kParts;
+  static constexpr int kParts = kDim >= 256 ? 16 : (kDim >= 64 ? 8 : 4);   // threads a column of S
+  static constexpr int kCols = 16;                        // value columns a block
+  static constexpr int kThreads = kCols * kParts;
   static constexpr int kRows = kDim / kParts;             // rows of S a thread holds
-  static constexpr int kSeg = kRows + 4;                  // a part's stretch of k (or q) in the staging buffer: the parts'
-                                                          // 16-byte reads fall into different banks
   static constexpr int kVecs = kChannel ? 3 : 2;          // vectors of kDim numbers staged a token: k | q (| decay - 1)
   static constexpr int kChunk = kDim <= 128 ? 16 : 8;     // tokens staged at a time (even)
+  static constexpr int kTail = kVecs * kDim;              // where what is not a vector of kDim numbers begins
+  // words staged a token: vectors | decay - 1, write strength, k . q, pad | the block's values
+  static constexpr int words(int value_bytes) { return kTail + 4 + kCols * value_bytes / 4; }
 };
 
 template <typename T, int kDim, bool kChannel>
 __global__ void __launch_bounds__(DeltaShape<kDim, kChannel>::kThreads)
-delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const T* __restrict__ v,
-                            long long ldv, const float* __restrict__ decay, const float* __restrict__ beta,
-                            float* __restrict__ out, float* __restrict__ state, long long state_stride,
-                            const int* __restrict__ cu_q, const int* __restrict__ state_slots, int heads, int kv_heads,
-                            int vdim) {
+delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ qk_dot,
+                            const T* __restrict__ v, long long ldv, const float* __restrict__ decay,
+                            const float* __restrict__ beta, float* __restrict__ out, float* __restrict__ state,
+                            long long state_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
+                            int heads, int kv_heads, int vdim) {
   typedef DeltaShape<kDim, kChannel> Shape;
-  constexpr int kParts = Shape::kParts, kThreads = Shape::kThreads, kRows = Shape::kRows, kSeg = Shape::kSeg;
-  constexpr int kVecs = Shape::kVecs, kChunk = Shape::kChunk;
-  constexpr int kVWords = 32 * sizeof(T) / 4;             // the block's 32 values of a token, in 32-bit words
-  constexpr int kTail = kVecs * kParts * kSeg;            // where what is not a vector of kDim numbers begins
-  constexpr int kTok = kTail + 4 + kVWords;               // words staged a token: vectors | decay - 1, write strength, pad | values
-  constexpr int kCopies = kVecs * (kDim / 4) + 2 + kVWords;   // asynchronous copies a token
+  constexpr int kParts = Shape::kParts, kThreads = Shape::kThreads, kRows = Shape::kRows;
+  constexpr int kChunk = Shape::kChunk, kCols = Shape::kCols, kPairs = kRows / 2, kTail = Shape::kTail;
+  constexpr int kVWords = kCols * sizeof(T) / 4;          // the block's values of a token, in 32-bit words
+  constexpr int kTok = Shape::words(sizeof(T));
   extern __shared__ __align__(16) float stage[];          // [2][kChunk][kTok]
   wait_for_prior_kernels();
   launch_dependents();
   const int r = blockIdx.x, h = blockIdx.y;
-  const int tid = threadIdx.x, part = tid % kParts, cl = tid / kParts, col0 = blockIdx.z * 32, col = col0 + cl;
+  const int tid = threadIdx.x, part = tid % kParts, cl = tid / kParts, col0 = blockIdx.z * kCols, col = col0 + cl;
   const int lo = cu_q[r], hi = cu_q[r + 1];
   const int slot = state_slots[r];
   if (hi <= lo || slot < 0) return;
   const int kh = h / (heads / kv_heads);
   const bool live = col < vdim;
-  float* Sg = state + slot * state_stride + (static_cast<long long>(h) * kDim + part * kRows) * vdim;
-  float S[kRows];
+  float* Sg = state + slot * state_stride + static_cast<long long>(h) * kDim * vdim + col;
+  // S[i]: rows row_of(i) and row_of(i) + 1
+  auto row_of = [&](int i) { return 4 * (part + kParts * (i >> 1)) + 2 * (i & 1); };
+  float2 S[kPairs];
 #pragma unroll
-  for (int i = 0; i < kRows; ++i) S[i] = live ? Sg[static_cast<long long>(i) * vdim + col] : 0.0f;
+  for (int i = 0; i < kPairs; ++i) {
+    const float* at = Sg + static_cast<long long>(row_of(i)) * vdim;
+    S[i] = live ? make_float2(at[0], at[vdim]) : make_float2(0.0f, 0.0f);
+  }
   // the copies of the chunk that starts at token t0, into buffer b: straight from memory into shared memory, so that
-  // they are under way while the chunk before is computed
+  // they are under way while the chunk before is computed.  A thread copies the same piece of every kStep-th token.
+  constexpr int kPieces = kDim / 4, kStep = kThreads / kPieces;
+  constexpr int kVStep = kThreads / kVWords;
+  const int c_tok = tid / kPieces, c_at = (tid % kPieces) * 4;
+  const int v_tok = tid / kVWords, v_word = tid % kVWords;
+  const bool v_there = col0 + v_word * (4 / static_cast<int>(sizeof(T))) < vdim;
+  const T* v_src = v + static_cast<long long>(h) * vdim + col0 + v_word * (4 / static_cast<int>(sizeof(T)));
   auto issue = [&](int t0, int b) {
     const int n_tok = min(kChunk, hi - t0);
-    for (int i = tid; i < n_tok * kCopies; i += kThreads) {
-      const int tok = i / kCopies, c = i - tok * kCopies;
-      const int t = t0 + tok;
-      float* dst = stage + (b * kChunk + tok) * kTok;
-      if (c < kVecs * (kDim / 4)) {
-        const int which = c / (kDim / 4);                        // 0: k, 1: q, 2: the decay a channel
-        const int e = (c - which * (kDim / 4)) * 4;              // element of it
-        const float* src = which == 2 ? decay + (static_cast<long long>(t) * heads + h) * kDim + e
-                                      : (which == 1 ? qn : kn) + (static_cast<long long>(t) * kv_heads + kh) * kDim + e;
-        async_copy_16(dst + which * kParts * kSeg + (e / kRows) * kSeg + e % kRows, src);
-      } else if (c < kVecs * (kDim / 4) + 2) {
-        const int which = c - kVecs * (kDim / 4);
-        if (which == 1 || !kChannel)
-          async_copy_4(dst + kTail + which, (which ? beta : decay) + static_cast<long long>(t) * heads + h);
-      } else {
-        const int w = c - kVecs * (kDim / 4) - 2;                // word w holds 4 / sizeof(T) values
-        const int first_col = col0 + w * (4 / static_cast<int>(sizeof(T)));
-        if (first_col < vdim)
-          async_copy_4(dst + kTail + 4 + w,
-                       v + static_cast<long long>(t) * ldv + static_cast<long long>(h) * vdim + first_col);
+    float* base = stage + b * kChunk * kTok;
+#pragma unroll
+    for (int tok = c_tok; tok < kChunk; tok += kStep) {
+      if (tok < n_tok) {
+        float* dst = base + tok * kTok + c_at;
+        const long long at = (static_cast<long long>(t0 + tok) * kv_heads + kh) * kDim + c_at;
+        async_copy_16(dst, kn + at);
+        async_copy_16(dst + kDim, qn + at);
+        if constexpr (kChannel)
+          async_copy_16(dst + 2 * kDim, decay + (static_cast<long long>(t0 + tok) * heads + h) * kDim + c_at);
       }
+    }
+#pragma unroll
+    for (int tok = v_tok; tok < kChunk; tok += kVStep)
+      if (tok < n_tok && v_there) async_copy_4(base + tok * kTok + kTail + 4 + v_word, v_src + (t0 + tok) * ldv);
+    const int tok = tid >> 2, which = tid & 3;               // 0: decay - 1, 1: write strength, 2: k . q
+    if (tok < n_tok && which < 3 && !(kChannel && which == 0)) {
+      const long long at = static_cast<long long>(t0 + tok) * heads + h;
+      async_copy_4(base + tok * kTok + kTail + which,
+                   which == 2 ? qk_dot + static_cast<long long>(t0 + tok) * kv_heads + kh : (which ? beta : decay) + at);
     }
     async_copies_commit();
   };
   // a token's numbers from the staging buffer into registers, one token ahead of the arithmetic
-  struct Tok { float k[kRows], q[kRows], g[kChannel ? kRows : 1], b, v; };
-  auto load = [&](Tok& x, const float* cur) {
+  struct Tok { float2 k[kPairs], q[kPairs], g[kChannel ? kPairs : 1]; float b, kq, v; };
+  auto load_vec = [&](float2* dst, const float* src) {
 #pragma unroll
-    for (int i = 0; i < kRows; i += 4) {
-      const float4 k4 = *reinterpret_cast<const float4*>(cur + part * kSeg + i);
-      const float4 q4 = *reinterpret_cast<const float4*>(cur + kParts * kSeg + part * kSeg + i);
-      x.k[i] = k4.x; x.k[i + 1] = k4.y; x.k[i + 2] = k4.z; x.k[i + 3] = k4.w;
-      x.q[i] = q4.x; x.q[i + 1] = q4.y; x.q[i + 2] = q4.z; x.q[i + 3] = q4.w;
-      if constexpr (kChannel) {
-        const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kParts * kSeg + part * kSeg + i);
-        x.g[i] = g4.x; x.g[i + 1] = g4.y; x.g[i + 2] = g4.z; x.g[i + 3] = g4.w;
-      }
+    for (int i = 0; i < kPairs; i += 2) {
+      const float4 f = *reinterpret_cast<const float4*>(src + 2 * kParts * i + 4 * part);
+      dst[i] = make_float2(f.x, f.y);
+      dst[i + 1] = make_float2(f.z, f.w);
     }
-    if constexpr (!kChannel) x.g[0] = cur[kTail];
+  };
+  auto load = [&](Tok& x, const float* cur) {
+    load_vec(x.k, cur);
+    load_vec(x.q, cur + kDim);
+    if constexpr (kChannel) {
+      load_vec(x.g, cur + 2 * kDim);
+    } else {
+      x.g[0] = make_float2(cur[kTail], cur[kTail]);
+    }
     x.b = cur[kTail + 1];
+    x.kq = cur[kTail + 2];
     x.v = to_float<T>(reinterpret_cast<const T*>(cur + kTail + 4)[cl]);
   };
-  auto reduce = [&](float x) {
-    x += __shfl_xor_sync(0xffffffffu, x, 1);
-    x += __shfl_xor_sync(0xffffffffu, x, 2);
-    if (kParts >= 8) x += __shfl_xor_sync(0xffffffffu, x, 4);
-    if (kParts >= 16) x += __shfl_xor_sync(0xffffffffu, x, 8);
-    return x;
-  };
   auto compute = [&](const Tok& x, int t) {
-    if constexpr (kChannel) {
+    // two chains a product; the parts' sums of both products go through the shuffles side by side
+    float2 a0 = make_float2(0.0f, 0.0f), a1 = a0, b0 = a0, b1 = a0;
 #pragma unroll
-      for (int i = 0; i < kRows; ++i) S[i] = fmaf(x.g[i], S[i], S[i]);
+    for (int i = 0; i < kPairs; i += 2) {
+      S[i] = fma2(x.g[kChannel ? i : 0], S[i], S[i]);            // g S, formed as S + (g - 1) S
+      S[i + 1] = fma2(x.g[kChannel ? i + 1 : 0], S[i + 1], S[i + 1]);
+      a0 = fma2(S[i], x.k[i], a0);
+      a1 = fma2(S[i + 1], x.k[i + 1], a1);
+      b0 = fma2(S[i], x.q[i], b0);
+      b1 = fma2(S[i + 1], x.q[i + 1], b1);
     }
-    float a0 = 0.0f, a1 = 0.0f;
+    float a = (a0.x + a1.x) + (a0.y + a1.y), b = (b0.x + b1.x) + (b0.y + b1.y);
 #pragma unroll
-    for (int i = 0; i < kRows; i += 2) {
-      a0 = fmaf(S[i], x.k[i], a0);
-      a1 = fmaf(S[i + 1], x.k[i + 1], a1);
+    for (int m = 1; m < kParts; m <<= 1) {
+      const float pa = __shfl_xor_sync(0xffffffffu, a, m), pb = __shfl_xor_sync(0xffffffffu, b, m);
+      a += pa;
+      b += pb;
     }
-    const float dot = reduce(a0 + a1);
-    const float u = x.b * (x.v - (kChannel ? dot : fmaf(x.g[0], dot, dot)));
-    float o0 = 0.0f, o1 = 0.0f;
+    const float u = x.b * (x.v - a);
+    const float2 uu = make_float2(u, u);
 #pragma unroll
-    for (int i = 0; i < kRows; i += 2) {
-      S[i] = fmaf(x.k[i], u, kChannel ? S[i] : fmaf(x.g[0], S[i], S[i]));
-      S[i + 1] = fmaf(x.k[i + 1], u, kChannel ? S[i + 1] : fmaf(x.g[0], S[i + 1], S[i + 1]));
-      o0 = fmaf(S[i], x.q[i], o0);
-      o1 = fmaf(S[i + 1], x.q[i + 1], o1);
-    }
-    const float o = reduce(o0 + o1);
-    if (live && part == 0) out[(static_cast<long long>(t) * heads + h) * vdim + col] = o;
+    for (int i = 0; i < kPairs; ++i) S[i] = fma2(x.k[i], uu, S[i]);
+    if (live && part == 0) out[(static_cast<long long>(t) * heads + h) * vdim + col] = fmaf(x.kq, u, b);
   };
   issue(lo, 0);
   async_copies_wait();
@@ -555,12 +601,18 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
     const float* base = stage + buf * kChunk * kTok;
     Tok x0, x1;
     load(x0, base);
-    for (int tok = 0; tok < n_tok; tok += 2) {
-      if (tok + 1 < n_tok) load(x1, base + (tok + 1) * kTok);
-      compute(x0, t0 + tok);
-      if (tok + 1 < n_tok) {
-        if (tok + 2 < n_tok) load(x0, base + (tok + 2) * kTok);
+    if (n_tok == kChunk) {                                       // no branch a token: loads and sums of neighbours overlap
+#pragma unroll 2
+      for (int tok = 0; tok < kChunk; tok += 2) {
+        load(x1, base + (tok + 1) * kTok);
+        compute(x0, t0 + tok);
+        load(x0, base + min(tok + 2, kChunk - 1) * kTok);        // (the last one is not used)
         compute(x1, t0 + tok + 1);
+      }
+    } else {
+      for (int tok = 0; tok < n_tok; ++tok) {
+        load(x0, base + tok * kTok);
+        compute(x0, t0 + tok);
       }
     }
     async_copies_wait();
@@ -569,7 +621,11 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
   }
   if (live) {
 #pragma unroll
-    for (int i = 0; i < kRows; ++i) Sg[static_cast<long long>(i) * vdim + col] = S[i];
+    for (int i = 0; i < kPairs; ++i) {
+      float* at = Sg + static_cast<long long>(row_of(i)) * vdim;
+      at[0] = S[i].x;
+      at[vdim] = S[i].y;
+    }
   }
 }
 
@@ -767,32 +823,39 @@ extern "C" int pih_causal_conv(int dtype, const void* x, long long ldx, const vo
 
 // The gated delta rule over a step's rows.  qkv [rows, ld]: q heads, k heads, v heads (after convolution and SiLU);
 // b [rows, ldb]: write-strength logits a head; a [rows, lda] (a_dtype): decay logits, one a head or (channels) one a head and
-// key channel, with decay_bias of the same layout; decay_log [heads].  scratch: fp32, rows * (2 * kv_heads * dim + heads +
-// heads * (channels ? dim : 1)), 16-byte aligned.  out: fp32 [rows, heads, vdim].  The state S [heads, dim, vdim] lies at the
+// key channel, with decay_bias of the same layout; decay_log [heads].  scratch: fp32, rows * (2 * kv_heads * dim + kv_heads +
+// heads + heads * (channels ? dim : 1)), 16-byte aligned.  out: fp32 [rows, heads, vdim].  The state S [heads, dim, vdim] lies at the
 // start of a request's slot.
 template <typename T, int D, bool CH>
-static void launch_delta_reg(cudaStream_t s, const float* qn, const float* kn, const T* v, long long ld, const float* decay,
+static void launch_delta_reg(cudaStream_t s, const float* qn, const float* kn, const float* qk_dot, const T* v, long long ld, const float* decay,
                              const float* beta, float* out, float* state, long long state_stride, const int* cu_q,
                              const int* state_slots, int requests, int heads, int kv_heads, int vdim) {
   typedef DeltaShape<D, CH> Shape;
-  const size_t staged = 2 * static_cast<size_t>(Shape::kChunk) *
-                        (Shape::kVecs * Shape::kParts * Shape::kSeg + 4 + 32 * sizeof(T) / 4) * sizeof(float);
-  if (staged > 48 * 1024)
+  const size_t needed = 2 * static_cast<size_t>(Shape::kChunk) * Shape::words(sizeof(T)) * sizeof(float);
+  const dim3 grid(requests, heads, (vdim + Shape::kCols - 1) / Shape::kCols);
+  // The chain from token to token is what a prompt costs: with no more blocks than SMs, every block asks for more than half
+  // of an SM's shared memory and so gets an SM alone.
+  const bool alone = static_cast<long long>(grid.x) * grid.y * grid.z <= 148;
+  const size_t staged = alone && needed < 116 * 1024 ? 116 * 1024 : needed;
+  static size_t raised = 48 * 1024;                            // (per instance)
+  if (staged > raised) {
     cudaFuncSetAttribute(delta_recurrence_reg_kernel<T, D, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                          static_cast<int>(staged));
-  launch_kernel(delta_recurrence_reg_kernel<T, D, CH>, dim3(requests, heads, (vdim + 31) / 32), dim3(Shape::kThreads), staged, s,
-                qn, kn, v, ld, decay, beta, out, state, state_stride, cu_q, state_slots, heads, kv_heads, vdim);
+    raised = staged;
+  }
+  launch_kernel(delta_recurrence_reg_kernel<T, D, CH>, grid,
+                dim3(Shape::kThreads), staged, s, qn, kn, qk_dot, v, ld, decay, beta, out, state, state_stride, cu_q, state_slots, heads, kv_heads, vdim);
 }
 
 template <typename T, bool CH>
-static int launch_delta(cudaStream_t s, const float* qn, const float* kn, const T* v, long long ld, const float* decay,
+static int launch_delta(cudaStream_t s, const float* qn, const float* kn, const float* qk_dot, const T* v, long long ld, const float* decay,
                         const float* beta, float* out, float* state, long long state_stride, const int* cu_q,
                         const int* state_slots, int requests, int heads, int kv_heads, int dim, int vdim) {
   const bool words = sizeof(T) == 4 || (ld % 2 == 0 && vdim % 2 == 0 && (reinterpret_cast<uintptr_t>(v) & 3) == 0);
   switch (words ? dim : 0) {                                   // (values are copied in 32-bit words)
 #define PIH_DELTA_REG(D)                                                                                               \
   case D:                                                                                                              \
-    launch_delta_reg<T, D, CH>(s, qn, kn, v, ld, decay, beta, out, state, state_stride, cu_q, state_slots, requests,   \
+    launch_delta_reg<T, D, CH>(s, qn, kn, qk_dot, v, ld, decay, beta, out, state, state_stride, cu_q, state_slots, requests,   \
                                heads, kv_heads, vdim);                                                                 \
     break
     PIH_DELTA_REG(16);
@@ -825,28 +888,31 @@ extern "C" int pih_gated_delta_rule(int dtype, const void* qkv, long long ld, co
                                     int kv_heads, int dim, int vdim, float unit_eps, float q_scale, void* stream) {
   if (rows <= 0 || requests <= 0) return 0;
   if (heads % kv_heads) return PIH_ERR_BAD_ARGUMENT;
-  if (heads > 65535 || (vdim + 31) / 32 > 65535) return PIH_ERR_UNSUPPORTED;
+  if (heads > 65535 || (vdim + 15) / 16 > 65535) return PIH_ERR_UNSUPPORTED;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const long long qk_size = static_cast<long long>(kv_heads) * dim;
   float* qn = static_cast<float*>(scratch);
   float* kn = qn + rows * qk_size;
   float* decay = kn + rows * qk_size;
   float* beta = decay + static_cast<long long>(rows) * heads * (channels ? dim : 1);
+  float* qk_dot = beta + static_cast<long long>(rows) * heads;
+  const int numbers = heads * (channels ? dim : 1);
+  const int parts = numbers > kDecaySlice ? 1 + (numbers + kDecaySlice - 1) / kDecaySlice : 1;
 #define PIH_DELTA(T, TA)                                                                                               \
   do {                                                                                                                 \
-    launch_kernel(delta_prepare_kernel<T, TA>, dim3(rows), dim3(128), 0, s, static_cast<const T*>(qkv), ld,            \
+    launch_kernel(delta_prepare_kernel<T, TA>, dim3(rows, parts), dim3(128), 0, s, static_cast<const T*>(qkv), ld,            \
                   static_cast<const T*>(b), ldb, static_cast<const TA*>(a), lda, channels,                             \
-                  static_cast<const float*>(decay_log), static_cast<const float*>(decay_bias), qn, kn, decay, beta,    \
-                  heads, kv_heads, dim, unit_eps, q_scale);                                                            \
+                  static_cast<const float*>(decay_log), static_cast<const float*>(decay_bias), qn, kn, qk_dot, decay,  \
+                  beta, heads, kv_heads, dim, unit_eps, q_scale);                                                            \
     PIH_LAUNCH_CHECK();                                                                                                \
     const T* v = static_cast<const T*>(qkv) + 2 * qk_size;                                                             \
     float* o = static_cast<float*>(out);                                                                               \
     float* st = static_cast<float*>(state);                                                                            \
     const int* cu = static_cast<const int*>(cu_q);                                                                     \
     const int* slots = static_cast<const int*>(state_slots);                                                           \
-    return channels ? launch_delta<T, true>(s, qn, kn, v, ld, decay, beta, o, st, state_stride, cu, slots, requests,   \
+    return channels ? launch_delta<T, true>(s, qn, kn, qk_dot, v, ld, decay, beta, o, st, state_stride, cu, slots, requests,   \
                                             heads, kv_heads, dim, vdim)                                                \
-                    : launch_delta<T, false>(s, qn, kn, v, ld, decay, beta, o, st, state_stride, cu, slots, requests,  \
+                    : launch_delta<T, false>(s, qn, kn, qk_dot, v, ld, decay, beta, o, st, state_stride, cu, slots, requests,  \
                                              heads, kv_heads, dim, vdim);                                              \
   } while (0)
   if (dtype == PIH_F32 && a_dtype == PIH_F32) PIH_DELTA(float, float);

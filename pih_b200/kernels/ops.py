@@ -732,7 +732,7 @@ class CudaOps:
         per_row = heads * (key_dim if channels else 1)
         assert qkv.stride(1) == 1 and beta.stride(1) == 1 and decay.stride(1) == 1 and beta.dtype == qkv.dtype
         assert beta.shape[1] >= heads and decay.shape[1] >= per_row and decay_bias.numel() == per_row
-        scratch = torch.empty(T * (2 * kv_heads * key_dim + heads + per_row), dtype=torch.float32, device=qkv.device)
+        scratch = torch.empty(T * (2 * kv_heads * key_dim + kv_heads + heads + per_row), dtype=torch.float32, device=qkv.device)
         out = torch.empty(T, heads, value_dim, dtype=torch.float32, device=qkv.device)
         rc = self.lib.pih_gated_delta_rule(_DT[qkv.dtype], _ptr(qkv), c_ll(qkv.stride(0)), _ptr(beta), c_ll(beta.stride(0)),
                                            _DT[decay.dtype], _ptr(decay), c_ll(decay.stride(0)), 1 if channels else 0,
