@@ -130,8 +130,8 @@ class GatedDeltaSpec:
 @dataclass(frozen=True)
 class SelectiveScanSpec:
     """Selective scan: ``inner`` channels of ``state`` numbers each.  Two branches read the block's input; the one passes
-    a short causal convolution (with a bias) and SiLU and drives the recurrence ``S[c, n] <- exp(dt_c A[c, n]) S[c, n] +
-    dt_c x_c B_n``, ``y_c = sum_n S[c, n] C_n + D_c x_c`` with ``A = -exp(A_log)``, whose B, C and (through ``dt_rank``
+    a short causal convolution (with a bias) and SiLU and drives the recurrence of a row of states per channel, ``row <- exp(dt A) * row
+    + (dt x) B``, ``y = <row, C> + D x`` with ``A = -exp(A_log)`` a row a channel, whose B, C and (through ``dt_rank``
     numbers) step sizes ``dt = softplus(.)`` are projections of it; SiLU of the other multiplies the output."""
     hidden: int
     inner: int

@@ -2,11 +2,11 @@
 
 ``W_in`` gives two branches ``[x | z]`` of ``inner`` channels.  x passes a short causal convolution per channel (with a
 bias) and SiLU; ``W_x`` of it gives ``[dt: dt_rank | B: state | C: state]``, ``W_dt`` the step-size logits of the channels.
-Then, per channel c and state n, with ``S`` starting at zero::
+Then, for every channel, with its row of states starting at zero::
 
-    dt = softplus(logit + bias)        A = -exp(A_log)
-    S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n
-    y_c = sum_n S[c, n] C_n + D_c x_c
+    dt  = softplus(logit + bias)       A = -exp(A_log)            (one step size, a row of rates)
+    row <- exp(dt * A) * row + (dt * x) B                         (element by element)
+    y   = <row, C> + D x
 
 and the output is ``W_o (y * silu(z))``.  (The recurrence of Gu and Dao, "Mamba: Linear-Time Sequence Modeling with
 Selective State Spaces".)  Step sizes, exponentials and the state are 32-bit whatever the compute dtype.  The state slot

@@ -41,8 +41,7 @@ def _errors(got, truth):
 
 
 def _check(got, truth, dtype, what, rounding=None):
-    """Per position: the error of the logits (mean taken off, root mean square over the vocabulary) relative to the
-    logits' spread.  32-bit: every position.  bfloat16, over the positions of all requests together: the median within
+    """Per position: how far the logits are off, up to a constant (root mean square), relative to the logits' spread.  32-bit: every position.  bfloat16, over the positions of all requests together: the median within
     rounding, and at most one position in ten beyond three times that.  ``rounding``: a function that gives the errors of
     a plain bfloat16 evaluation of the same steps (torch operations with a rounding after each), for a model so steep that
     rounding alone exceeds the fixed bound."""
