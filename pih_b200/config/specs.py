@@ -144,14 +144,102 @@ class SelectiveScanSpec:
 
 
 @dataclass(frozen=True)
+class StateSpaceSpec:
+    """State-space duality (Mamba-2): per head a matrix state ``S [state, value_dim]`` with one decay a token,
+    ``S <- exp(-exp(A) dt) S + dt B x^T``, ``y = S^T C + D x``.  ``W_in`` gives ``[z | x | B | C | dt]``; x, B and C pass one
+    short causal convolution (with a bias) and SiLU; B and C have ``groups`` heads shared by groups of heads;
+    ``dt = softplus(. + bias)``.  The output ``y silu(z)`` is RMS-normed in ``norm_groups`` equal parts, each by its own
+    root mean square (``norm_eps``), with a weight a column."""
+    hidden: int
+    heads: int
+    value_dim: int
+    state: int
+    groups: int
+    norm_groups: int
+    conv_taps: int
+    norm_eps: float
+    kind: str = "state_space"
+    names: Mapping[str, str] = _names(w_in="mix.in", conv="mix.conv", conv_bias="mix.conv.b", dt_bias="mix.dt_bias",
+                                      a_log="mix.A_log", skip="mix.D", out_norm="mix.norm", o="mix.o")
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.value_dim
+
+    @property
+    def bc_size(self) -> int:
+        """Columns of B (and of C)."""
+        return self.groups * self.state
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """Gated linear attention: per head a matrix state ``S [key_dim, value_dim]`` whose rows decay by a number of their own,
+    ``S <- diag(a) S + k v^T``, read out ``S^T q`` with q times ``key_dim ** -0.5``.  The decays ``a = sigmoid(z) ** (1 /
+    temperature)`` come through a narrow projection of ``decay_rank`` numbers (``decay_down``, then ``decay_up`` with a
+    bias).  The read-out of a head is RMS-normed over ``value_dim`` (one weight for all heads) and multiplied by ``silu`` of
+    a gate projection."""
+    hidden: int
+    heads: int
+    key_dim: int
+    value_dim: int
+    decay_rank: int
+    temperature: float
+    norm_eps: float
+    kind: str = "gated_linear"
+    names: Mapping[str, str] = _names(q="mix.q", k="mix.k", v="mix.v", gate="mix.g", o="mix.o", out_norm="mix.norm",
+                                      decay_down="mix.a1", decay_up="mix.a2", decay_bias="mix.a2.b")
+
+    @property
+    def qk_size(self) -> int:
+        return self.heads * self.key_dim
+
+    @property
+    def v_size(self) -> int:
+        return self.heads * self.value_dim
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory with exponential gates (the mLSTM of xLSTM): per head ``S [key_dim, value_dim]``, a key sum ``n [key_dim]``
+    and a running maximum ``m``.  With the log gates ``i = cap tanh((. + b_i) / cap)`` and ``f = logsigmoid(cap tanh((. + b_f) /
+    cap))``: ``m' = max(f + m, i)``, ``S <- exp(f + m - m') S + exp(i - m') k v^T``, n likewise with k alone; the read-out
+    ``S^T q / (max(|n . q|, exp(-m')) + floor)`` with q times ``key_dim ** -0.5``.  It is divided by its root mean square a
+    head (``norm_eps``), multiplied by a weight a column of all heads and by ``sigmoid`` of a gate projection."""
+    hidden: int
+    heads: int
+    key_dim: int
+    value_dim: int
+    gate_cap: float
+    norm_eps: float
+    floor: float = 1e-6
+    kind: str = "matrix_memory"
+    names: Mapping[str, str] = _names(q="mix.q", k="mix.k", v="mix.v", gate="mix.g", o="mix.o", out_norm="mix.norm",
+                                      write="mix.i", write_bias="mix.i.b", keep="mix.f", keep_bias="mix.f.b")
+
+    @property
+    def qk_size(self) -> int:
+        return self.heads * self.key_dim
+
+    @property
+    def v_size(self) -> int:
+        return self.heads * self.value_dim
+
+
+@dataclass(frozen=True)
 class ParallelSpec:
     """Two mixers side by side that read the same input: ``left_scale * left(x) + right_scale * right(x)``.  The specs'
-    tensor names are below the block's prefix as anywhere.  At most one of the two may ask for a paged cache."""
+    tensor names are below the block's prefix as anywhere.  At most one of the two may ask for a paged cache.
+
+    ``out_norm_eps`` not None: each output is RMS-normed over the width with a weight of its own (the tensors
+    ``names["left"]`` and ``names["right"]``) before it is scaled and added."""
     left: object
     right: object
     left_scale: float = 1.0
     right_scale: float = 1.0
+    out_norm_eps: Optional[float] = None
     kind: str = "parallel"
+    names: Mapping[str, str] = _names(left="mix.left.out", right="mix.right.out")
 
     @property
     def hidden(self) -> int:
@@ -235,12 +323,14 @@ class ComputedRopeSpec:
     ``(i, i + rotary_dim / 2)`` or, with ``interleaved``, the neighbours ``(2i, 2i + 1)``.  ``stretch`` = (factor, low,
     high, original) slows the slow pairs down: with ``turns_i = original f_i / (2 pi)`` (how often pair i goes round
     within ``original`` positions) and ``t_i = clamp((turns_i - low) / (high - low), 0, 1)``, the frequency becomes
-    ``f_i (t_i + (1 - t_i) / factor)`` — untouched from ``high`` turns on, divided by ``factor`` up to ``low`` turns."""
+    ``f_i (t_i + (1 - t_i) / factor)`` — untouched from ``high`` turns on, divided by ``factor`` up to ``low`` turns.
+    ``slowdown`` divides every frequency (linear scaling)."""
     head_dim: int
     rotary_dim: int
     theta: float
     interleaved: bool = False
     stretch: Optional[Sequence[float]] = None
+    slowdown: float = 1.0
     kind: str = "rope_computed"
 
 
@@ -339,7 +429,7 @@ class ScoredMoESpec:
     ``experts`` real experts and behind them ``identity`` experts without tensors whose output is the input itself.
     The choice goes by ``score + correction`` (a learned vector), restricted to the ``groups_keep`` best of
     ``groups`` equal groups of neighbouring outputs (a group's score: its largest choice score); the ``top`` chosen
-    outputs weigh with their scores, as they are (``renormalize`` False) or divided by their sum.  ``shared``: a
+    outputs weigh with their scores, as they are (``renormalize`` False) or divided by their sum, times ``weight_scale``.  ``shared``: a
     gated feed-forward that runs for every row and is added, multiplied by ``sigmoid`` of a one-row projection
     (``shared_gate`` False: added as it is; its spec may be any feed-forward's).
 
@@ -362,6 +452,7 @@ class ScoredMoESpec:
     gated: bool = True
     weigh: str = "output"
     shared_gate: bool = True
+    weight_scale: float = 1.0
     kind: str = "scored_moe"
     names: Mapping[str, str] = _names(router="mlp.router", correction="mlp.correction", expert="mlp.e{}.", gate="gate",
                                       up="up", down="down", shared_gate="mlp.shared.sg")
@@ -410,7 +501,10 @@ class WindowAttentionSpec:
     * ``softcap``: the scaled score becomes ``softcap * tanh(score / softcap)``;
     * ``chunk`` > 0: a row sees only the keys of its own chunk of that many places, counted from place 0 of the sequence
       (``window`` 0 beside it: all of the chunk's keys up to the row);
-    * ``head_gate``: head h's output is multiplied by ``sigmoid`` of a one-row projection of the mixer's input."""
+    * ``head_gate``: head h's output is multiplied by ``sigmoid`` of a one-row projection of the mixer's input;
+    * ``column_gate``: the concatenated heads are multiplied by ``sigmoid`` of a projection of the mixer's input, column by
+      column;
+    * ``biases``: the projections of q, k and v and the output projection have biases."""
     hidden: int
     heads: int
     kv_heads: int
@@ -435,10 +529,13 @@ class WindowAttentionSpec:
     # ``window``); None: ``window``
     cache_window: Optional[int] = None
     chunk: int = 0
+    column_gate: bool = False
+    biases: bool = False
     kind: str = "window_attention"
     names: Mapping[str, str] = _names(q="mix.q", k="mix.k", v="mix.v", o="mix.o", q_norm="mix.q.norm", k_norm="mix.k.norm",
                                       q_conv="mix.q.conv", k_conv="mix.k.conv", v_conv="mix.v.conv", bias="mix.rel",
-                                      sink="mix.sink", gate="mix.g")
+                                      sink="mix.sink", gate="mix.g", q_bias="mix.q.b", k_bias="mix.k.b", v_bias="mix.v.b",
+                                      o_bias="mix.o.b")
 
     @property
     def q_size(self) -> int:
@@ -467,7 +564,10 @@ class BlockSpec:
     """One layer: ``h += mixer(norm_in(h)); h += ffn(norm_post(h))`` for
     ``arrangement == "prenorm"``; ``h += norm_in(mixer(h)); h += norm_post(ffn(h))``
     for ``arrangement == "outnorm"`` (the norms sit on the sub-layers' outputs,
-    the sub-layers read the stream itself); ``arrangement == "hyper"``: the pre-norm
+    the sub-layers read the stream itself); ``h += s1 * norm_in_out(mixer(norm_in(h)));
+    h += s2 * norm_post_out(ffn(norm_post(h)))`` for ``arrangement == "sandwich"`` (a norm before
+    and behind each sub-layer; with ``layer_scale`` the vectors s1, s2 are tensors, else they are
+    absent); ``arrangement == "hyper"``: the pre-norm
     layer over several streams (``hyper``); ``ffn`` and ``norm_post`` None: the layer has
     no feed-forward.  ``residual_scale`` multiplies what a "prenorm" layer's
     sub-layers add to the stream.  ``prefix`` is the layer's tensor-name prefix in the
@@ -482,6 +582,11 @@ class BlockSpec:
                                       norm_post="post_attention_layernorm.")
     hyper: Optional[HyperSpec] = None
     residual_scale: float = 1.0
+    # "sandwich": the norms behind the mixer and behind the feed-forward (``names``: "norm_in_out", "norm_post_out"), and
+    # whether a vector multiplies each normed output (``names``: "scale_in", "scale_post")
+    norm_in_out: Optional[object] = None
+    norm_post_out: Optional[object] = None
+    layer_scale: bool = False
 
 
 @dataclass(frozen=True)
@@ -532,6 +637,8 @@ class ModelSpec:
     streams: int = 0
     # the logits are the head's product times this number
     logit_scale: float = 1.0
+    # the logits become ``cap * tanh(logits / cap)``; None: as they are
+    logit_softcap: Optional[float] = None
     bigram: Optional[BigramSpec] = None
     # the embedding output is the table's row times this number (a 32-bit stream)
     embed_scale: float = 1.0
@@ -563,3 +670,7 @@ class ModelSpec:
         if any(b.residual_scale != 1.0 and (b.arrangement != "prenorm" or self.stream_dtype != "float32")
                for b in self.blocks):
             raise ValueError("residual_scale goes with pre-norm layers on a 32-bit stream")
+        if any(b.arrangement == "sandwich" for b in self.blocks) and self.stream_dtype != "float32":
+            raise ValueError("layers with norms before and behind their sub-layers keep a 32-bit stream")
+        if self.logit_softcap is not None and self.logit_softcap <= 0:
+            raise ValueError("logit_softcap must be positive")

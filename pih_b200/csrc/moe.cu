@@ -77,10 +77,11 @@ moe_route_kernel(const float* __restrict__ logits, int rows, int experts, int to
 // the choice goes by s + correction, among the outputs of the
 // ``keep`` best of ``groups`` equal groups of neighbours (a group's score: its largest choice score; the others count
 // as minus infinity); the ``top`` largest are chosen (ties: the smaller index) and weigh with their s, divided by the
-// chosen ones' sum only with ``renormalize``.  One warp a row; ``flags``: [warps][groups] ints of shared memory.
+// chosen ones' sum only with ``renormalize``, and times ``weight_scale``.  One warp a row; ``flags``: [warps][groups] ints of shared memory.
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction, int rows,
-                        int experts, int top, int groups, int keep, int renormalize, int scoring, int* __restrict__ expert_of,
+                        int experts, int top, int groups, int keep, int renormalize, int scoring, float weight_scale,
+                        int* __restrict__ expert_of,
                         float* __restrict__ weight_of, int* __restrict__ rank_of, int* __restrict__ counts,
                         int* __restrict__ pos_of) {
   extern __shared__ float route_smem[];
@@ -173,8 +174,9 @@ moe_route_scored_kernel(const float* __restrict__ logits, long long ld, const fl
     }
   }
   __syncwarp();
-  if (renormalize)
-    for (int k = lane; k < top; k += 32) weight_of[static_cast<long long>(row) * top + k] /= chosen_sum;
+  const float fix = weight_scale / (renormalize ? chosen_sum + 1e-20f : 1.0f);
+  if (fix != 1.0f)
+    for (int k = lane; k < top; k += 32) weight_of[static_cast<long long>(row) * top + k] *= fix;
 }
 
 // plan: [0 .. experts] first position of an expert's rows; [experts+1 .. 2 experts+1] first tile of an expert.
@@ -540,8 +542,8 @@ extern "C" int pih_moe_route(const void* logits, int rows, int experts, int top,
 // The same outputs as pih_moe_route from the scored routing (see moe_route_scored_kernel); logits fp32 [rows, ld] of which
 // the first ``experts`` columns are the router's outputs; correction fp32 [experts] or null.
 extern "C" int pih_moe_route_scored(const void* logits, long long ld, const void* correction, int rows, int experts, int top,
-                                    int groups, int keep, int renormalize, int scoring, void* ints, void* weight_of,
-                                    int grouped, void* stream) {
+                                    int groups, int keep, int renormalize, int scoring, float weight_scale, void* ints,
+                                    void* weight_of, int grouped, void* stream) {
   if (rows <= 0) return 0;
   if (experts < 1 || experts > 1024 || top < 1 || top > experts || groups < 1 || groups > 1024 || experts % groups ||
       keep < 1 || keep > groups)
@@ -556,7 +558,7 @@ extern "C" int pih_moe_route_scored(const void* logits, long long ld, const void
   int* plan = counts + experts;
   launch_kernel(moe_route_scored_kernel, dim3((rows + 3) / 4), dim3(128), 4 * 2 * groups * sizeof(float), s,
                 static_cast<const float*>(logits), ld, static_cast<const float*>(correction), rows, experts, top, groups,
-                keep, renormalize, scoring, expert_of, static_cast<float*>(weight_of), rank_of,
+                keep, renormalize, scoring, weight_scale, expert_of, static_cast<float*>(weight_of), rank_of,
                 grouped ? counts : static_cast<int*>(nullptr), pos_of);
   PIH_LAUNCH_CHECK();
   if (!grouped) return 0;

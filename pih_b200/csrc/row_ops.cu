@@ -9,6 +9,7 @@
 //   gate_mul        a * sigmoid(g) or a * silu(g), the gate a strided view
 //   unary_act       relu(z + bias)^2 or the error-function form of GELU of z + bias
 //   scale_rows      x *= s in place (32-bit)
+//   softcap_rows    x = cap tanh(x / cap) in place (32-bit)
 #include "common.cuh"
 
 namespace pih {
@@ -225,6 +226,13 @@ __global__ void scale_rows_kernel(float* __restrict__ x, long long n, float s) {
   if (i < n) x[i] *= s;
 }
 
+__global__ void softcap_rows_kernel(float* __restrict__ x, long long n, float cap) {
+  wait_for_prior_kernels();
+  launch_dependents();
+  const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
 }  // namespace pih
 
 using namespace pih;
@@ -345,6 +353,15 @@ extern "C" int pih_scale_rows(void* x, long long n, float scale, void* stream) {
   if (n <= 0) return 0;
   launch_kernel(scale_rows_kernel, flat_grid(n), dim3(256), 0, static_cast<cudaStream_t>(stream), static_cast<float*>(x), n,
                 scale);
+  PIH_LAUNCH_CHECK();
+  return 0;
+}
+
+extern "C" int pih_softcap_rows(void* x, long long n, float cap, void* stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.0f)) return PIH_ERR_BAD_ARGUMENT;
+  launch_kernel(softcap_rows_kernel, flat_grid(n), dim3(256), 0, static_cast<cudaStream_t>(stream), static_cast<float*>(x), n,
+                cap);
   PIH_LAUNCH_CHECK();
   return 0;
 }

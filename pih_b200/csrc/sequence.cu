@@ -3,12 +3,16 @@
 //   embedding_stream      table rows (bf16 or fp32) times one number -> a 32-bit stream
 //   rmsnorm_stream        h (fp32) += scale * (delta + bias) (+ the token's embedding and a vector: a loop's next pass);
 //                         out = h / sqrt(mean(h^2) + eps) * w, w a vector or ONE number
+//   stream_norm_norm      h (fp32) += rms(y + bias) * w1, or with a pair of outputs h += rms(rms(y + bias) * wl + rms(y2 + bias2) *
+//                         wr) * w1; out = rms(h) * w2: a norm behind a sub-layer, the sum and the next norm in one pass
 //   causal_conv           short causal convolution per channel over each request's rows, the last taps-1 inputs
 //                         carried in the request's state slot
 //   delta_prepare         unit-norm q and k per head, decay (one a head, or one a head and key channel) and write
 //                         strength per head (32-bit)
 //   delta_recurrence      gated delta rule: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
-//   gated_rmsnorm         per-head RMS norm of the read-out, times a weight, times silu(gate) or sigmoid(gate)
+//   gated_rmsnorm         per-head RMS norm of the read-out (divided by a number a head first), times a weight, times silu(gate)
+//                         or sigmoid(gate)
+//   gated_part_rmsnorm    y * silu(gate), then an RMS norm in equal parts of the row with a weight a column
 //   rglru_gates, _chain   real-gated linear recurrent unit: S <- a S + sqrt(1 - a^2) (i u), out = S * gelu(y)
 //
 // A step's rows are packed: request r owns rows cu_q[r] .. cu_q[r+1]-1 in the order of their positions, and
@@ -195,6 +199,130 @@ rmsnorm_stream_kernel(float* __restrict__ h, const StreamAdd<TD> add, const floa
     if (rows == nullptr) load_floats<V>(v, hr + c);            // (the thread's own store)
     else stream_sum<TD, V>(v, hr, dr, er, add, c);
     write(v, c);
+  }
+}
+
+// Two sums over a block of up to 1024 threads at once, in an order that depends on blockDim only.
+__device__ __forceinline__ float2 block_sum_pair(float2 v, float2* scratch /* 33 */) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  __syncthreads();
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  if (warp == 0) {
+    float2 t = lane < warps ? scratch[lane] : make_float2(0.0f, 0.0f);
+    t.x = warp_sum(t.x);
+    t.y = warp_sum(t.y);
+    if (lane == 0) scratch[32] = t;
+  }
+  __syncthreads();
+  return scratch[32];
+}
+
+// What a sub-layer gave, on its way through the norm behind it: y (+ bias) or a pair of outputs, each RMS-normed with a weight
+// of its own and added.
+template <typename TD>
+struct NormedOutput {
+  const TD* y;
+  const float* bias;                                           // null: none
+  const TD* y2;                                                // null: no pair
+  const float* bias2;
+  const float* weight_left;
+  const float* weight_right;
+  float pair_eps;
+  const float* weight;                                         // of the norm behind the sub-layer
+  float eps;
+};
+
+// One block a row, V columns a thread at a time, up to kNormHeld pieces a thread, all in registers.  With ``rows`` nothing
+// is stored back and ``out`` holds the gathered rows.
+constexpr int kNormHeld = 4;
+template <typename TD, typename TO, int V>
+__global__ void __launch_bounds__(1024)
+stream_norm_norm_kernel(float* __restrict__ h, const NormedOutput<TD> add, const float* __restrict__ weight,
+                        TO* __restrict__ out, const int* __restrict__ rows, int width, float eps) {
+  __shared__ float2 scratch[33];
+  wait_for_prior_kernels();
+  launch_dependents();
+  const int row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
+  float* hr = h + static_cast<long long>(row) * width;
+  const TD* yr = add.y + static_cast<long long>(row) * width;
+  const TD* yr2 = add.y2 != nullptr ? add.y2 + static_cast<long long>(row) * width : nullptr;
+  const int step = static_cast<int>(blockDim.x) * V, c0 = static_cast<int>(threadIdx.x) * V;
+  const float n = static_cast<float>(width);
+  float u[kNormHeld][V], v[kNormHeld][V];
+  float2 ss = make_float2(0.0f, 0.0f);
+  auto with_bias = [&](float (&x)[V], const float* bias, int c) {
+    if (bias != nullptr) {
+      float b[V];
+      load_floats<V>(b, bias + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[i] += b[i];
+    }
+  };
+#pragma unroll
+  for (int k = 0; k < kNormHeld; ++k) {
+    const int c = c0 + k * step;
+    if (c >= width) continue;
+    load_floats<V>(u[k], yr + c);
+    with_bias(u[k], add.bias, c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss.x = fmaf(u[k][i], u[k][i], ss.x);
+    if (yr2 != nullptr) {
+      load_floats<V>(v[k], yr2 + c);
+      with_bias(v[k], add.bias2, c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss.y = fmaf(v[k][i], v[k][i], ss.y);
+    }
+  }
+  ss = block_sum_pair(ss, scratch);
+  if (yr2 != nullptr) {
+    const float left = 1.0f / sqrtf(ss.x / n + add.pair_eps), right = 1.0f / sqrtf(ss.y / n + add.pair_eps);
+    ss = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (int k = 0; k < kNormHeld; ++k) {
+      const int c = c0 + k * step;
+      if (c >= width) continue;
+      float wl[V], wr[V];
+      load_floats<V>(wl, add.weight_left + c);
+      load_floats<V>(wr, add.weight_right + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        u[k][i] = fmaf(v[k][i] * right, wr[i], u[k][i] * left * wl[i]);
+        ss.x = fmaf(u[k][i], u[k][i], ss.x);
+      }
+    }
+    ss = block_sum_pair(ss, scratch);
+  }
+  const float behind = 1.0f / sqrtf(ss.x / n + add.eps);
+  ss = make_float2(0.0f, 0.0f);
+#pragma unroll
+  for (int k = 0; k < kNormHeld; ++k) {
+    const int c = c0 + k * step;
+    if (c >= width) continue;
+    float w[V];
+    load_floats<V>(w, add.weight + c);
+    load_floats<V>(v[k], hr + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      v[k][i] = fmaf(u[k][i] * behind, w[i], v[k][i]);
+      ss.x = fmaf(v[k][i], v[k][i], ss.x);
+    }
+    if (rows == nullptr) store_floats<V>(hr + c, v[k]);
+  }
+  ss = block_sum_pair(ss, scratch);
+  const float scale = 1.0f / sqrtf(ss.x / n + eps);
+  TO* o = out + static_cast<long long>(blockIdx.x) * width;
+#pragma unroll
+  for (int k = 0; k < kNormHeld; ++k) {
+    const int c = c0 + k * step;
+    if (c >= width) continue;
+    float w[V];
+    load_floats<V>(w, weight + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[k][i] = v[k][i] * scale * w[i];
+    store_floats<V>(o + c, v[k]);
   }
 }
 
@@ -449,15 +577,6 @@ __global__ void delta_recurrence_kernel(const float* __restrict__ qn, const floa
 // so no load from memory and only one barrier a chunk lie on the chain from token to token; a token's numbers go from there
 // to registers one token ahead.  The order of the additions is fixed by the kernel, not by the step's make-up or by where a
 // chunk begins.  With kChannel the decay (as g - 1, [rows, heads, kDim]) multiplies the rows of S; it is staged like k and q.
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 d;
-  asm("{\n\t.reg .b64 ra, rb, rc, rd;\n\t"
-      "mov.b64 ra, {%2, %3};\n\tmov.b64 rb, {%4, %5};\n\tmov.b64 rc, {%6, %7};\n\t"
-      "fma.rn.f32x2 rd, ra, rb, rc;\n\tmov.b64 {%0, %1}, rd;\n\t}"
-      : "=f"(d.x), "=f"(d.y)
-      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-  return d;
-}
 __device__ __forceinline__ void async_copy_16(void* smem_dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst))), "l"(src));
 }
@@ -630,12 +749,13 @@ delta_recurrence_reg_kernel(const float* __restrict__ qn, const float* __restric
 }
 
 // One warp a (row, head): o fp32 [rows, heads, vdim]; gate [rows, ldg] and out [rows, ldo] with head h at column h * vdim.
-// activation 0: silu(gate), 1: sigmoid(gate); out_scale multiplies.
+// activation 0: silu(gate), 1: sigmoid(gate); out_scale multiplies.  divisor: fp32 [rows, heads] or null, divides o before the
+// norm; head_weight: how far the weights of two heads lie apart (0: one weight for all heads).
 template <typename TG, typename T>
 __global__ void __launch_bounds__(128)
 gated_rmsnorm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, long long ldg, const float* __restrict__ weight,
                      T* __restrict__ out, long long ldo, long long rows_heads, int heads, int vdim, float eps, int activation,
-                     float out_scale) {
+                     float out_scale, const float* __restrict__ divisor, int head_weight) {
   wait_for_prior_kernels();
   launch_dependents();
   const long long item = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -644,16 +764,62 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, l
   const long long row = item / heads;
   const int h = static_cast<int>(item % heads);
   const float* src = o + item * vdim;
+  const float share = divisor != nullptr ? 1.0f / divisor[item] : 1.0f;
+  weight += static_cast<long long>(h) * head_weight;
   float ss = 0.0f;
-  for (int i = lane; i < vdim; i += 32) ss = fmaf(src[i], src[i], ss);
+  for (int i = lane; i < vdim; i += 32) {
+    const float x = src[i] * share;
+    ss = fmaf(x, x, ss);
+  }
   ss = warp_sum(ss);
-  const float scale = 1.0f / sqrtf(ss / static_cast<float>(vdim) + eps) * out_scale;
+  const float scale = share / sqrtf(ss / static_cast<float>(vdim) + eps) * out_scale;
   const TG* g = gate + row * ldg + static_cast<long long>(h) * vdim;
   T* dst = out + row * ldo + static_cast<long long>(h) * vdim;
   for (int i = lane; i < vdim; i += 32) {
     const float z = to_float<TG>(g[i]);
     dst[i] = from_float<T>(src[i] * scale * weight[i] * ((activation == 1 ? 1.0f : z) / (1.0f + expf(-z))));
   }
+}
+
+// Block (row, part): y fp32 [rows, width] times silu(gate [rows, ldg]), the part's own RMS norm, a weight a column.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_part_rmsnorm_kernel(const float* __restrict__ y, const T* __restrict__ gate, long long ldg,
+                          const float* __restrict__ weight, T* __restrict__ out, long long ldo, int width, int part,
+                          float eps, float out_scale) {
+  __shared__ float scratch[33];
+  wait_for_prior_kernels();
+  launch_dependents();
+  constexpr int kHeld = 4;
+  const long long row = blockIdx.x;
+  const int c0 = blockIdx.y * part;
+  const float* yr = y + row * width + c0;
+  const T* gr = gate + row * ldg + c0;
+  auto gated = [&](int i) {
+    const float z = to_float<T>(gr[i]);
+    return yr[i] * (z / (1.0f + expf(-z)));
+  };
+  float held[kHeld];
+  float ss = 0.0f;
+#pragma unroll
+  for (int k = 0; k < kHeld; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    held[k] = i < part ? gated(i) : 0.0f;
+    ss = fmaf(held[k], held[k], ss);
+  }
+  for (int i = threadIdx.x + kHeld * blockDim.x; i < part; i += blockDim.x) {
+    const float v = gated(i);
+    ss = fmaf(v, v, ss);
+  }
+  ss = block_sum(ss, scratch);
+  const float scale = out_scale / sqrtf(ss / static_cast<float>(part) + eps);
+  T* o = out + row * ldo + c0;
+#pragma unroll
+  for (int k = 0; k < kHeld; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i < part) o[i] = from_float<T>(held[k] * scale * weight[c0 + i]);
+  }
+  for (int i = threadIdx.x + kHeld * blockDim.x; i < part; i += blockDim.x) o[i] = from_float<T>(gated(i) * scale * weight[c0 + i]);
 }
 
 // The unit in two kernels.  rglru_gates (a thread a (row, channel), every row at once): from the gate logits
@@ -791,6 +957,50 @@ extern "C" int pih_rmsnorm_stream(int delta_dtype, int out_dtype, void* h, const
   return 0;
 }
 
+// h [.., width] fp32: h += rms(y + bias) * add_weight (add_eps), or with y2 the pair in y's place (see NormedOutput), then out =
+// rms(h) * weight (eps).  y, y2 [.., width] of delta_dtype; bias, bias2 nullable; the weights fp32 [width].
+extern "C" int pih_stream_norm_norm(int delta_dtype, int out_dtype, void* h, const void* y, const void* bias, const void* y2,
+                                    const void* bias2, const void* weight_left, const void* weight_right, float pair_eps,
+                                    const void* add_weight, float add_eps, const void* weight, float eps, void* out,
+                                    const void* rows, int n_out, int width, void* stream) {
+  if (n_out <= 0) return 0;
+  if (y == nullptr || add_weight == nullptr || weight == nullptr ||
+      (y2 != nullptr && (weight_left == nullptr || weight_right == nullptr)))
+    return PIH_ERR_BAD_ARGUMENT;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool four = width % 4 == 0 && aligned(h) && aligned(y) && aligned(bias) && aligned(y2) && aligned(bias2) &&
+                    aligned(weight_left) && aligned(weight_right) && aligned(add_weight) && aligned(weight) && aligned(out);
+  const int pieces = four ? width / 4 : width;
+  int threads = pieces <= 512 ? (pieces + 31) / 32 * 32 : 512;
+  if (pieces > threads * kNormHeld) threads = 1024;
+  if (pieces > threads * kNormHeld) return PIH_ERR_UNSUPPORTED;
+#define PIH_NN_V(TD, TO, V)                                                                                           \
+  do {                                                                                                                \
+    NormedOutput<TD> add;                                                                                             \
+    add.y = static_cast<const TD*>(y);                                                                                \
+    add.bias = static_cast<const float*>(bias);                                                                       \
+    add.y2 = static_cast<const TD*>(y2);                                                                              \
+    add.bias2 = static_cast<const float*>(bias2);                                                                     \
+    add.weight_left = static_cast<const float*>(weight_left);                                                         \
+    add.weight_right = static_cast<const float*>(weight_right);                                                       \
+    add.pair_eps = pair_eps;                                                                                          \
+    add.weight = static_cast<const float*>(add_weight);                                                               \
+    add.eps = add_eps;                                                                                                \
+    launch_kernel(stream_norm_norm_kernel<TD, TO, V>, dim3(n_out), dim3(threads), 0, s, static_cast<float*>(h), add,   \
+                  static_cast<const float*>(weight), static_cast<TO*>(out), static_cast<const int*>(rows), width, eps); \
+  } while (0)
+#define PIH_NN(TD, TO)                                                                                                \
+  do { if (four) PIH_NN_V(TD, TO, 4); else PIH_NN_V(TD, TO, 1); } while (0)
+  if (delta_dtype == PIH_F32 && out_dtype == PIH_F32) PIH_NN(float, float);
+  else if (delta_dtype == PIH_BF16 && out_dtype == PIH_BF16) PIH_NN(bf16, bf16);
+  else return PIH_ERR_BAD_ARGUMENT;
+#undef PIH_NN
+#undef PIH_NN_V
+  PIH_LAUNCH_CHECK();
+  return 0;
+}
+
 extern "C" int pih_causal_conv(int dtype, const void* x, long long ldx, const void* w, const void* in_bias,
                                const void* out_bias, void* out, long long ldo, int channels, int taps, int activation,
                                void* state, long long state_stride, long long state_offset, const void* cu_q,
@@ -922,23 +1132,48 @@ extern "C" int pih_gated_delta_rule(int dtype, const void* qkv, long long ld, co
 #undef PIH_DELTA
 }
 
-// o fp32 [rows, heads, vdim]; gate [rows, ldg] (gate_dtype), out [rows, ldo] (dtype); activation 0: SiLU, 1: sigmoid.
+// o fp32 [rows, heads, vdim]; gate [rows, ldg] (gate_dtype), out [rows, ldo] (dtype); activation 0: SiLU, 1: sigmoid; divisor
+// fp32 [rows, heads] or null; head_weight 0: weight [vdim], else weight [heads, head_weight].
 extern "C" int pih_gated_rmsnorm(int dtype, int gate_dtype, const void* o, const void* gate, long long ldg,
                                  const void* weight, void* out, long long ldo, int rows, int heads, int vdim, float eps,
-                                 int activation, float out_scale, void* stream) {
+                                 int activation, float out_scale, const void* divisor, int head_weight, void* stream) {
   if (rows <= 0) return 0;
-  if (activation < 0 || activation > 1) return PIH_ERR_BAD_ARGUMENT;
+  if (activation < 0 || activation > 1 || (head_weight != 0 && head_weight < vdim)) return PIH_ERR_BAD_ARGUMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const long long items = static_cast<long long>(rows) * heads;
   dim3 grid(static_cast<unsigned>((items + 3) / 4));
 #define PIH_GN(TG, T)                                                                                                  \
   launch_kernel(gated_rmsnorm_kernel<TG, T>, grid, dim3(128), 0, s, static_cast<const float*>(o), static_cast<const TG*>(gate), \
-                ldg, static_cast<const float*>(weight), static_cast<T*>(out), ldo, items, heads, vdim, eps, activation, out_scale)
+                ldg, static_cast<const float*>(weight), static_cast<T*>(out), ldo, items, heads, vdim, eps, activation, out_scale, \
+                static_cast<const float*>(divisor), head_weight)
   if (dtype == PIH_F32 && gate_dtype == PIH_F32) PIH_GN(float, float);
   else if (dtype == PIH_BF16 && gate_dtype == PIH_BF16) PIH_GN(bf16, bf16);
   else if (dtype == PIH_BF16 && gate_dtype == PIH_F32) PIH_GN(float, bf16);
   else return PIH_ERR_BAD_ARGUMENT;
 #undef PIH_GN
+  PIH_LAUNCH_CHECK();
+  return 0;
+}
+
+// y fp32 [rows, width] contiguous; gate [rows, ldg], out [rows, ldo] of ``dtype``; ``parts`` equal stretches of the row are
+// normed each by itself after the gate
+extern "C" int pih_gated_part_rmsnorm(int dtype, const void* y, const void* gate, long long ldg, const void* weight, void* out,
+                                      long long ldo, int rows, int width, int parts, float eps, float out_scale,
+                                      void* stream) {
+  if (rows <= 0) return 0;
+  if (parts < 1 || width < 1 || width % parts) return PIH_ERR_BAD_ARGUMENT;
+  if (parts > 65535) return PIH_ERR_UNSUPPORTED;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int part = width / parts;
+  const int threads = part >= 1024 ? 256 : (part >= 256 ? 128 : (part >= 64 ? 64 : 32));
+#define PIH_GPN(T)                                                                                                     \
+  launch_kernel(gated_part_rmsnorm_kernel<T>, dim3(rows, parts), dim3(threads), 0, s, static_cast<const float*>(y),      \
+                static_cast<const T*>(gate), ldg, static_cast<const float*>(weight), static_cast<T*>(out), ldo, width,  \
+                part, eps, out_scale)
+  if (dtype == PIH_F32) PIH_GPN(float);
+  else if (dtype == PIH_BF16) PIH_GPN(bf16);
+  else return PIH_ERR_BAD_ARGUMENT;
+#undef PIH_GPN
   PIH_LAUNCH_CHECK();
   return 0;
 }

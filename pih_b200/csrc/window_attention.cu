@@ -1,5 +1,5 @@
 // Softmax attention over a sliding window or inside chunks of places, with optional kept first tokens, a sink in the
-// denominator, a learned bias by distance, capped scores and a gate a head.
+// denominator, a learned bias by distance, capped scores and a gate a head or a column.
 //
 // The cache holds one vector per token, [k: kv_heads x dim | v: kv_heads x vdim], in pages: cache[page][offset][width].
 // A row at position p sees the keys j <= p with p - j < window (window 0: all) and j / chunk == p / chunk (chunk 0: all;
@@ -7,9 +7,9 @@
 //
 //   score  = (q . k) scale;  cap > 0: cap tanh(score / cap);  bias: + bias[head][min(p - j, distances - 1)]
 //   weight = exp(score) / (sum over the seen keys of exp(score) + exp(sink[head]))        (sink null: no such term)
-//   out    = sum weight v, times sigmoid(gate[row][head]) where there is a gate, times one number
+//   out    = sum weight v, times sigmoid(gate[row][head]) (or gate[row][head, column]) where there is a gate, times one number
 //
-//   window_qk_prepare        per row: RMS norm over the WHOLE q (and k) projection with a weight a column, rotation of the
+//   window_qk_prepare        per row: the projections' biases, where they have any; RMS norm over the WHOLE q (and k) projection with a weight a column, rotation of the
 //                            first columns of every head in neighbouring pairs or in halves, by a table of (cos, sin) or
 //                            by angles position * f_i computed in 32-bit from frequencies; without write_kv the rows
 //                            hold q alone and nothing goes to the cache (a mixer that reads another's keys and values);
@@ -41,6 +41,7 @@ struct WindowRule {
   const float* bias;     // [heads][distances] or null
   int distances;
   float out_scale;       // multiplies the output
+  int gate_columns;      // columns of the gate a head: 0: one number a head, else vdim of them
   // the first key that a row at ``pos`` sees (apart from the kept ones); grows with ``pos``
   __device__ __forceinline__ int first_of(int pos) const {
     int first = window > 0 ? max(0, pos - window + 1) : 0;
@@ -92,7 +93,8 @@ __device__ __forceinline__ float element_of_words(const uint32_t (&w)[WORDS], in
 // element.
 template <typename T>
 __global__ void __launch_bounds__(256)
-window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict__ q_out, const float* __restrict__ q_norm,
+window_qk_prepare_kernel(const T* __restrict__ src, long long ld, const float* __restrict__ in_bias,
+                         T* __restrict__ q_out, const float* __restrict__ q_norm,
                          const float* __restrict__ k_norm, float eps, const float* __restrict__ table,
                          const float* __restrict__ freq, int rot,
                          int interleaved, int max_positions, const int* __restrict__ positions,
@@ -121,6 +123,11 @@ window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict_
     if (slot < 0) return;
     const T* v = values_from_keys ? x + nq : x + nq + nk;
     T* dst = cache + slot * width + nk;
+    if (in_bias != nullptr) {
+      const float* b = in_bias + (values_from_keys ? nq : nq + nk);
+      for (int e = threadIdx.x; e < nv; e += blockDim.x) dst[e] = from_float<T>(to_float<T>(v[e]) + b[e]);
+      return;
+    }
     if (aligned && nv % V == 0) {
       for (int e = threadIdx.x * V; e < nv; e += blockDim.x * V)
         *reinterpret_cast<uint4*>(dst + e) = *reinterpret_cast<const uint4*>(v + e);
@@ -141,6 +148,7 @@ window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict_
   const T* xp = part == 0 ? x : x + nq;
   const int n = part == 0 ? nq : nk;
   const float* w = part == 0 ? q_norm : k_norm;
+  const float* b_in = in_bias == nullptr ? nullptr : (part == 0 ? in_bias : in_bias + nq);
   T* dst = part == 0 ? q_out + row * nq : (slot >= 0 ? cache + slot * width : nullptr);
   if (dst == nullptr) return;
   if (turns && cs == nullptr && half <= kTurnPairs) {
@@ -162,6 +170,7 @@ window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict_
 #pragma unroll
       for (int i = 0; i < V; ++i) {
         held[u][i] = element_of_words<T, kWords>(raw, i);
+        if (b_in != nullptr && e < n) held[u][i] += b_in[e + i];
         ss = fmaf(held[u][i], held[u][i], ss);
       }
     }
@@ -198,6 +207,7 @@ window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict_
 #pragma unroll
         for (int i = 0; i < V; ++i) {
           float p = element_of_words<T, kWords>(raw, i);
+          if (b_in != nullptr) p += b_in[pe + i];
           if (w != nullptr) p = p * inv * w[pe + i];
           float cosine, sine;
           if (cs != nullptr) { cosine = cs[2 * (pair0 + i)]; sine = cs[2 * (pair0 + i) + 1]; }
@@ -216,7 +226,7 @@ window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict_
   if (w != nullptr) {
     float ss = 0.0f;
     for (int e = threadIdx.x; e < n; e += blockDim.x) {
-      const float v = to_float<T>(xp[e]);
+      const float v = to_float<T>(xp[e]) + (b_in != nullptr ? b_in[e] : 0.0f);
       ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, scratch);
@@ -224,14 +234,14 @@ window_qk_prepare_kernel(const T* __restrict__ src, long long ld, T* __restrict_
   }
   for (int e = threadIdx.x; e < n; e += blockDim.x) {
     const int c = e % dim;                                     // column within the head
-    float o = to_float<T>(xp[e]);
+    float o = to_float<T>(xp[e]) + (b_in != nullptr ? b_in[e] : 0.0f);
     if (w != nullptr) o = o * inv * w[e];
     if (turns && c < rot) {
       int pair, other;
       bool first;                                              // whether e is the first number of its pair
       if (interleaved) { pair = c >> 1; first = (c & 1) == 0; other = first ? e + 1 : e - 1; }
       else { pair = c < half ? c : c - half; first = c < half; other = first ? e + half : e - half; }
-      float p = to_float<T>(xp[other]);
+      float p = to_float<T>(xp[other]) + (b_in != nullptr ? b_in[other] : 0.0f);
       if (w != nullptr) p = p * inv * w[other];
       float cosine, sine;
       if (cs != nullptr) { cosine = cs[2 * pair]; sine = cs[2 * pair + 1]; }
@@ -358,7 +368,7 @@ __device__ __forceinline__ void window_stretch(const float* q, const T* __restri
 // The sink joins the denominator, the sums are divided, the gate multiplies; a lane holds columns PL lane + e.
 template <typename T, int PL>
 __device__ __forceinline__ void window_finish(float (&a)[PL], float m, float l, const float* __restrict__ sink, int head,
-                                              const T* __restrict__ gate, float scale, int vdim, int lane,
+                                              const T* __restrict__ gate, bool gate_columns, float scale, int vdim, int lane,
                                               T* __restrict__ out,
                                               uint32_t* __restrict__ error) {
   float fix = 1.0f;
@@ -373,7 +383,13 @@ __device__ __forceinline__ void window_finish(float (&a)[PL], float m, float l, 
     l = 1.0f;
   }
   float f = fix / l * scale;
-  if (gate != nullptr) f *= 1.0f / (1.0f + expf(-to_float<T>(*gate)));
+  if (gate != nullptr && gate_columns) {
+#pragma unroll
+    for (int e = 0; e < PL; ++e)
+      if (PL * lane + e < vdim) a[e] *= 1.0f / (1.0f + expf(-to_float<T>(gate[PL * lane + e])));
+  } else if (gate != nullptr) {
+    f *= 1.0f / (1.0f + expf(-to_float<T>(*gate)));
+  }
 #pragma unroll
   for (int e = 0; e < PL; ++e)
     if (PL * lane + e < vdim) out[PL * lane + e] = from_float<T>(a[e] * f);
@@ -449,8 +465,8 @@ window_attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, lo
       p[2 + 32 * e + lane] = a[e];                             // (column PL lane + e; beyond vdim: zero)
     return;
   }
-  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head : nullptr, rule.out_scale, vdim, lane,
-                       o, error);
+  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head * max(rule.gate_columns, 1) : nullptr,
+                       rule.gate_columns > 0, rule.out_scale, vdim, lane, o, error);
 }
 
 // A warp a (row, head): the parts' sums folded in order, then the sink, the division and the gate.
@@ -458,7 +474,7 @@ template <typename T, int PL>
 __global__ void __launch_bounds__(128)
 window_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, long long ldo,
                               const int* __restrict__ request_of_row, const int* __restrict__ cu_q, int rows, int heads,
-                              int vdim, int splits, int small_rows, float out_scale,
+                              int vdim, int splits, int small_rows, float out_scale, int gate_columns,
                               const float* __restrict__ sink, const T* __restrict__ gate, long long ld_gate,
                               uint32_t* __restrict__ error) {
   wait_for_prior_kernels();
@@ -489,8 +505,8 @@ window_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
     for (int e = 0; e < PL; ++e)
       a[e] = fmaf(p[2 + 32 * e + lane], d, a[e]);
   }
-  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head : nullptr, out_scale, vdim, lane,
-                       out + row * ldo + static_cast<long long>(head) * vdim, error);
+  window_finish<T, PL>(a, m, l, sink, head, gate != nullptr ? gate + row * ld_gate + head * max(gate_columns, 1) : nullptr,
+                       gate_columns > 0, out_scale, vdim, lane, out + row * ldo + static_cast<long long>(head) * vdim, error);
 }
 
 // Tensor cores for requests of more than small_rows rows (bf16).  A block is kTileRows consecutive rows of one request and one
@@ -782,7 +798,20 @@ window_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16*
   const bool bad = (ra < nrows && (!(l_a > 0.0f) || l_a > 3.0e38f)) || (rb < nrows && (!(l_b > 0.0f) || l_b > 3.0e38f));
   if (bad) publish_error(error, kAttentionDenominator);
   float f_a = l_a > 0.0f ? fix_a / l_a * rule.out_scale : 0.0f, f_b = l_b > 0.0f ? fix_b / l_b * rule.out_scale : 0.0f;
-  if (gate != nullptr) {
+  if (gate != nullptr && rule.gate_columns > 0) {
+    const __nv_bfloat16* ga = gate + (row0 + ra) * ld_gate + static_cast<long long>(head) * vdim;
+    const __nv_bfloat16* gb = ga + 8 * ld_gate;
+#pragma unroll
+    for (int n = 0; n < VDIM / 8; ++n) {
+      const int col = n * 8 + 2 * (lane & 3);
+      if (col >= vdim) continue;
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        if (ra < nrows) O[n][c] *= __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(ga[col + c])));
+        if (rb < nrows) O[n][2 + c] *= __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(gb[col + c])));
+      }
+    }
+  } else if (gate != nullptr) {
     if (ra < nrows) f_a *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(row0 + ra) * ld_gate + head])));
     if (rb < nrows) f_b *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(row0 + rb) * ld_gate + head])));
   }
@@ -808,8 +837,8 @@ typedef __nv_bfloat16 bf16;
 // key columns as they are become the values); q_out [rows, heads x dim]; q_norm fp32 [heads x dim], k_norm fp32
 // [kv_heads x dim] or null; table fp32 [max_positions, rot / 2, 2] or null, and then freq fp32 [rot / 2] or null (angles
 // computed from the position); cache [num_pages, page_size, kv_heads (dim + vdim)].  write_kv 0: the rows hold q alone and
-// nothing goes to the cache.
-extern "C" int pih_window_qk_prepare(int dtype, const void* src, long long ld, void* q_out, const void* q_norm,
+// nothing goes to the cache.  in_bias: fp32, one number a column of src, or null.
+extern "C" int pih_window_qk_prepare(int dtype, const void* src, long long ld, const void* in_bias, void* q_out, const void* q_norm,
                                      const void* k_norm, float eps, const void* table, const void* freq, int rot,
                                      int interleaved, int max_positions, const void* positions, const void* slot_mapping,
                                      void* cache, int page_size, int num_pages, int rows, int heads, int kv_heads, int dim,
@@ -823,7 +852,7 @@ extern "C" int pih_window_qk_prepare(int dtype, const void* src, long long ld, v
   const int threads = heads * dim >= 1024 ? 256 : 128;
 #define PIH_WQK(T)                                                                                                     \
   launch_kernel(window_qk_prepare_kernel<T>, dim3(rows, write_kv ? 3 : 1), dim3(threads), 0, s,                        \
-                static_cast<const T*>(src), ld,                                                                        \
+                static_cast<const T*>(src), ld, static_cast<const float*>(in_bias),                                    \
                 static_cast<T*>(q_out), static_cast<const float*>(q_norm), static_cast<const float*>(k_norm), eps,     \
                 static_cast<const float*>(rot > 0 ? table : nullptr), static_cast<const float*>(rot > 0 ? freq : nullptr), \
                 rot, interleaved, max_positions,                                                                       \
@@ -866,7 +895,7 @@ extern "C" int pih_window_attention_tile_takes(int dim, int vdim) {
 // The attention of the step's rows: q [rows, heads x dim] (prepared), out [rows, ldo] (heads x vdim columns are written,
 // times out_scale).  bias fp32
 // [heads, distances] or null; sink fp32 [heads] or null; gate [rows, ld_gate] of the compute dtype (column h: head h's
-// logit) or null.  ``tile`` (bf16 only, sizes that pih_window_attention_tile_takes): requests of more than 16 rows run
+// logit; with gate_columns one logit a column of the output) or null.  ``tile`` (bf16 only, sizes that pih_window_attention_tile_takes): requests of more than 16 rows run
 // on the tensor-core kernel.  ``small``: the other rows (all rows without ``tile``) run on the warp kernel, their keys
 // cut into ``splits`` parts (1: uncut) through ``partial`` (fp32 [rows, heads, splits, 2 + 32 x the value columns a lane]).
 extern "C" int pih_window_attention(int dtype, const void* q, void* out, long long ldo, float out_scale,
@@ -874,7 +903,7 @@ extern "C" int pih_window_attention(int dtype, const void* q, void* out, long lo
                                     const void* q_start, int rows, int requests, int heads, int kv_heads, int dim, int vdim,
                                     int page_size, int num_pages, float scale, float cap, const void* bias, int distances,
                                     int window, int chunk, int keep_first, const void* sink, const void* gate, long long ld_gate,
-                                    int tile, int small, int splits, void* partial, void* error, void* stream) {
+                                    int gate_columns, int tile, int small, int splits, void* partial, void* error, void* stream) {
   if (rows <= 0) return 0;
   if (dim > 1024 || vdim > 32 * kWinMaxPerLane || heads % kv_heads || splits < 1) return PIH_ERR_UNSUPPORTED;
   if (tile && (dtype != PIH_BF16 || !pih_window_attention_tile_takes(dim, vdim) || ldo % 2)) return PIH_ERR_UNSUPPORTED;
@@ -887,6 +916,7 @@ extern "C" int pih_window_attention(int dtype, const void* q, void* out, long lo
   rule.chunk = chunk;
   rule.keep_first = window > 0 || chunk > 0 ? keep_first : 0;
   rule.out_scale = out_scale;
+  rule.gate_columns = gate_columns ? vdim : 0;
   rule.scale = scale;
   rule.cap = cap;
   rule.bias = static_cast<const float*>(bias);
@@ -920,7 +950,7 @@ extern "C" int pih_window_attention(int dtype, const void* q, void* out, long lo
     if (splits > 1)                                                                                                    \
       launch_kernel(window_attention_merge_kernel<T, PL>, dim3(grid.x), dim3(128), 0, s,                               \
                     static_cast<const float*>(partial), static_cast<T*>(out), ldo, static_cast<const int*>(request_of_row), \
-                    static_cast<const int*>(cu_q), rows, heads, vdim, splits, small_rows, rule.out_scale,              \
+                    static_cast<const int*>(cu_q), rows, heads, vdim, splits, small_rows, rule.out_scale, rule.gate_columns, \
                     static_cast<const float*>(sink), static_cast<const T*>(gate), ld_gate, static_cast<uint32_t*>(error)); \
   } while (0)
 #define PIH_WAG(T)                                                                                                     \

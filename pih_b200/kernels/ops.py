@@ -112,7 +112,8 @@ class CudaOps:
                      "pih_diff_qk_prepare", "pih_diff_attention", "pih_diff_attention_tile_takes", "pih_moe_route_scored",
                      "pih_act_mul", "pih_embed_positions", "pih_hyper_stream", "pih_window_qk_prepare",
                      "pih_window_attention", "pih_window_attention_tile_takes", "pih_embed_bigram", "pih_rmsnorm_rows",
-                     "pih_rotate_heads", "pih_gate_mul", "pih_unary_act", "pih_selective_scan", "pih_gemm_skinny_bias_gelu", "pih_scale_rows", "pih_moe_gather_scaled"):
+                     "pih_rotate_heads", "pih_gate_mul", "pih_unary_act", "pih_selective_scan", "pih_gemm_skinny_bias_gelu", "pih_scale_rows", "pih_moe_gather_scaled",
+                     "pih_softcap_rows", "pih_stream_norm_norm", "pih_gated_part_rmsnorm", "pih_linear_memory", "pih_memory_copies"):
             getattr(lib, name).restype = c_int
         lib.pih_attention_scratch_floats.restype = c_ll
         lib.pih_top_logprobs_scratch_words.restype = c_ll
@@ -648,6 +649,28 @@ class CudaOps:
         self._check(rc, "rmsnorm_stream")
         return out
 
+    def stream_norm_norm(self, h: torch.Tensor, y: torch.Tensor, add_weight: torch.Tensor, add_eps: float, weight: torch.Tensor,
+                         eps: float, bias: Optional[torch.Tensor] = None, pair: Optional[tuple] = None,
+                         rows: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+        """A norm behind a sub-layer, the sum and the next norm in one pass over the 32-bit stream: ``h += rms(y + bias) *
+        add_weight`` (stored back unless ``rows`` selects), then ``rms(h) * weight`` rounded to ``out_dtype``, with ``rms(x) =
+        x / sqrt(mean(x^2) + eps)``.  ``pair`` = (y2, bias2, left weight, right weight, eps): ``rms(y + bias) * left weight +
+        rms(y2 + bias2) * right weight``, kept in 32-bit, stands in the place of ``y + bias``.  Weights and biases fp32
+        ``[width]``."""
+        width = h.shape[-1]
+        assert h.dtype == torch.float32 and h.is_contiguous() and y.is_contiguous() and y.shape == h.shape
+        y2, bias2, left, right, pair_eps = pair if pair is not None else (None, None, None, None, 0.0)
+        assert y2 is None or (y2.is_contiguous() and y2.shape == h.shape and y2.dtype == y.dtype)
+        for t in (add_weight, weight, bias, bias2, left, right):
+            assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == (width,))
+        n_out = h.numel() // width if rows is None else rows.shape[0]
+        out = torch.empty((n_out, width), dtype=out_dtype, device=h.device)
+        rc = self.lib.pih_stream_norm_norm(_DT[y.dtype], _DT[out_dtype], _ptr(h), _ptr(y), _ptr(bias), _ptr(y2), _ptr(bias2),
+                                           _ptr(left), _ptr(right), c_float(pair_eps), _ptr(add_weight), c_float(add_eps),
+                                           _ptr(weight), c_float(eps), _ptr(out), _ptr(rows), n_out, width, self._stream())
+        self._check(rc, "stream_norm_norm")
+        return out
+
     def linear_batched(self, x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
                        rotate: Optional[dict] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``out[t, b] = x[t, b] . w[b]^T``: x ``[T, B, K]`` (a view whose rows may be strided), w ``[B, N, K]``;
@@ -745,20 +768,102 @@ class CudaOps:
         return out
 
     def gated_rmsnorm(self, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, activation: str = "silu",
-                      scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      scale: float = 1.0, out: Optional[torch.Tensor] = None,
+                      divisor: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``o / sqrt(mean(o^2) + eps) * weight * act(gate) * scale`` per (row, head): o fp32 ``[T, heads, vdim]``, gate
-        ``[T, heads * vdim]`` (a view), weight fp32 ``[vdim]``, ``activation`` "silu" or "sigmoid"; into ``out`` (a view,
-        ``[T, heads * vdim]``) or a new tensor of the gate's dtype, which is returned."""
+        ``[T, heads * vdim]`` (a view), weight fp32 ``[vdim]`` or ``[heads * vdim]``, ``activation`` "silu" or "sigmoid"; into
+        ``out`` (a view, ``[T, heads * vdim]``) or a new tensor of the gate's dtype, which is returned.  ``divisor`` (fp32
+        ``[T, heads]``): o is divided by it first."""
         T, heads, vdim = o.shape
+        assert weight.numel() in (vdim, heads * vdim) and (divisor is None or (divisor.is_contiguous()
+                                                                               and divisor.shape == (T, heads)))
         assert o.is_contiguous() and gate.stride(1) == 1 and gate.shape[1] >= heads * vdim
         if out is None:
             out = torch.empty(T, heads * vdim, dtype=gate.dtype, device=o.device)
         assert out.shape == (T, heads * vdim) and out.stride(1) == 1
         rc = self.lib.pih_gated_rmsnorm(_DT[out.dtype], _DT[gate.dtype], _ptr(o), _ptr(gate), c_ll(gate.stride(0)),
                                         _ptr(weight), _ptr(out), c_ll(out.stride(0)), T, heads, vdim, c_float(eps),
-                                        {"silu": 0, "sigmoid": 1}[activation], c_float(scale), self._stream())
+                                        {"silu": 0, "sigmoid": 1}[activation], c_float(scale), _ptr(divisor),
+                                        vdim if weight.numel() != vdim else 0, self._stream())
         self._check(rc, "gated_rmsnorm")
         return out
+
+    def gated_part_rmsnorm(self, y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,
+                           scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``y * silu(gate)`` (y fp32 ``[T, n]``, gate a view ``[T, n]``), then every one of ``parts`` equal stretches of the
+        row divided by its own root mean square (``eps`` inside the root), times ``weight`` (fp32 ``[n]``) and ``scale``; into
+        ``out`` (a view) or a new tensor of the gate's dtype."""
+        T, n = y.shape
+        assert y.is_contiguous() and gate.shape == (T, n) and gate.stride(1) == 1 and n % parts == 0
+        assert weight.dtype == torch.float32 and weight.shape == (n,)
+        if out is None:
+            out = torch.empty(T, n, dtype=gate.dtype, device=y.device)
+        assert out.shape == (T, n) and out.stride(1) == 1 and out.dtype == gate.dtype
+        rc = self.lib.pih_gated_part_rmsnorm(_DT[gate.dtype], _ptr(y), _ptr(gate), c_ll(gate.stride(0)), _ptr(weight),
+                                             _ptr(out), c_ll(out.stride(0)), T, n, parts, c_float(eps), c_float(scale),
+                                             self._stream())
+        self._check(rc, "gated_part_rmsnorm")
+        return out
+
+    # -- linear attention with a decaying matrix state -------------------------------------------------------------------
+    def memory_copies(self, value_dim: int) -> int:
+        """How many running maxima a head of ``matrix_memory`` keeps in its state."""
+        return self.lib.pih_memory_copies(value_dim)
+
+    def _linear_memory(self, gate_kind: int, q, k, v, *, gate0, gate1=None, bias0, bias1=None, A=None, constant=0.0, floor=0.0,
+                       q_scale=1.0, skip=None, divisor=None, state, step, heads, groups, key_dim, value_dim, what):
+        T = q.shape[0]
+        assert q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1 and q.dtype == k.dtype == v.dtype
+        assert q.shape[1] >= groups * key_dim and k.shape[1] >= groups * key_dim and v.shape[1] >= heads * value_dim
+        assert gate0.stride(1) == 1 and (gate1 is None or gate1.stride(1) == 1) and state.dtype == torch.float32
+        assert bias0.dtype == torch.float32 and (bias1 is None or bias1.dtype == torch.float32)
+        out = torch.empty(T, heads, value_dim, dtype=torch.float32, device=q.device)
+        rc = self.lib.pih_linear_memory(
+            _DT[q.dtype], gate_kind, _ptr(q), c_ll(q.stride(0)), _ptr(k), c_ll(k.stride(0)), _ptr(v), c_ll(v.stride(0)),
+            _ptr(gate0), c_ll(gate0.stride(0)), _ptr(gate1), c_ll(gate1.stride(0) if gate1 is not None else 0), _ptr(bias0),
+            _ptr(bias1), _ptr(A), c_float(constant), c_float(floor), c_float(q_scale), _ptr(skip), _ptr(out), _ptr(divisor),
+            _ptr(state), c_ll(state.stride(0)), _ptr(step.cu_q), _ptr(step.state_slots), T, step.num_requests, heads, groups,
+            key_dim, value_dim, self._stream())
+        self._check(rc, what)
+        return out
+
+    def gated_linear(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, *, bias: torch.Tensor,
+                     temperature: float, q_scale: float, state: torch.Tensor, step, heads: int, key_dim: int,
+                     value_dim: int) -> torch.Tensor:
+        """Gated linear attention over the step's rows from each request's state (``state[slot, :heads * key_dim *
+        value_dim]`` is S): ``a = sigmoid(z + bias) ** (1 / temperature)`` a head and key channel, ``S <- diag(a) S + k v^T``;
+        returns ``S^T q * q_scale``, fp32 ``[T, heads, value_dim]``.  q, k ``[T, heads * key_dim]``, v ``[T, heads * value_dim]``
+        (views), z fp32 ``[T, heads * key_dim]`` (a view), ``bias`` fp32."""
+        assert z.dtype == torch.float32 and z.shape[1] >= heads * key_dim and bias.numel() == heads * key_dim
+        return self._linear_memory(0, q, k, v, gate0=z, bias0=bias, constant=1.0 / temperature, q_scale=q_scale, state=state,
+                                   step=step, heads=heads, groups=heads, key_dim=key_dim, value_dim=value_dim,
+                                   what="gated_linear")
+
+    def state_space(self, C: torch.Tensor, B: torch.Tensor, x: torch.Tensor, dt: torch.Tensor, *, dt_bias: torch.Tensor,
+                    A: torch.Tensor, D: torch.Tensor, state: torch.Tensor, step, heads: int, groups: int, state_dim: int,
+                    value_dim: int) -> torch.Tensor:
+        """State-space duality over the step's rows: ``dt = softplus(dt + dt_bias)`` a head, ``S <- exp(A dt) S + dt B x^T``,
+        ``y = S^T C + D x``, fp32 ``[T, heads, value_dim]``.  B, C ``[T, groups * state_dim]`` (a group serves ``heads / groups``
+        heads in a row), x ``[T, heads * value_dim]``, dt ``[T, heads]`` (views of the compute dtype); ``dt_bias``, ``A``
+        (negative), ``D`` fp32 ``[heads]``."""
+        assert dt.dtype == x.dtype and dt.shape[1] >= heads and A.dtype == D.dtype == torch.float32
+        assert dt_bias.numel() == A.numel() == D.numel() == heads
+        return self._linear_memory(1, C, B, x, gate0=dt, bias0=dt_bias, A=A, skip=D, state=state, step=step, heads=heads,
+                                   groups=groups, key_dim=state_dim, value_dim=value_dim, what="state_space")
+
+    def matrix_memory(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, write: torch.Tensor, keep: torch.Tensor, *,
+                      write_bias: torch.Tensor, keep_bias: torch.Tensor, cap: float, floor: float, q_scale: float,
+                      state: torch.Tensor, step, heads: int, key_dim: int, value_dim: int):
+        """Matrix memory with exponential gates over the step's rows (logits ``write``, ``keep`` ``[T, heads]``, views of the
+        compute dtype; see ``MatrixMemorySpec``) from each request's state: S, then n ``[heads, key_dim]``, then
+        ``memory_copies`` running maxima a head.  Returns ``(S^T q * q_scale, the divisor)``, fp32 ``[T, heads, value_dim]``
+        and ``[T, heads]``."""
+        assert write.dtype == keep.dtype == q.dtype and write_bias.numel() == keep_bias.numel() == heads
+        divisor = torch.empty(q.shape[0], heads, dtype=torch.float32, device=q.device)
+        out = self._linear_memory(2, q, k, v, gate0=write, gate1=keep, bias0=write_bias, bias1=keep_bias, constant=cap,
+                                  floor=floor, q_scale=q_scale, divisor=divisor, state=state, step=step, heads=heads,
+                                  groups=heads, key_dim=key_dim, value_dim=value_dim, what="matrix_memory")
+        return out, divisor
 
     def selective_scan(self, u: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, z: torch.Tensor, *, dt_bias, A, D,
                        state: torch.Tensor, step, scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -896,7 +1001,7 @@ class CudaOps:
         ``routing`` selects the other router: scores are the softmax over all ``outputs`` (the first columns of
         ``logits``, whose rows may be longer), the choice goes by score plus ``correction`` within the
         ``groups_keep`` best of ``groups`` groups, the chosen weigh with their scores (``renormalize``: divided by
-        their sum), and the outputs behind the experts that have matrices are identity experts (the row itself).
+        their sum; times ``weight_scale``), and the outputs behind the experts that have matrices are identity experts (the row itself).
         ``routing["scoring"]`` "sigmoid": a score is the sigmoid of the output's own logit.  ``routing["gated"]`` False:
         an expert is ``W_down max(W_up x, 0)^2`` and ``w_gate_up`` is ``[experts, ff, hidden]``.  ``routing["weigh"]``
         "input": an expert reads the row times its weight (rounded to the compute dtype) and the outputs are summed
@@ -925,7 +1030,8 @@ class CudaOps:
             rc = self.lib.pih_moe_route_scored(_ptr(logits), c_ll(logits.stride(0)), _ptr(routing.get("correction")), T,
                                                experts, top, int(routing.get("groups", 1)), int(routing.get("groups_keep", 1)),
                                                1 if routing.get("renormalize") else 0,
-                                               {"softmax": 0, "sigmoid": 1}[routing.get("scoring", "softmax")], _ptr(ints),
+                                               {"softmax": 0, "sigmoid": 1}[routing.get("scoring", "softmax")],
+                                               c_float(routing.get("weight_scale", 1.0)), _ptr(ints),
                                                _ptr(weight_of), 0 if few else 1, self._stream())
         self._check(rc, "moe_route")
         self.launches += 0 if few else 2
@@ -1121,15 +1227,18 @@ class CudaOps:
     def window_qk_prepare(self, src: torch.Tensor, *, q_norm, k_norm, eps: float, rope_table, rotary_dim: int,
                           interleaved: bool, positions, slot_mapping, cache: torch.Tensor, heads: int, kv_heads: int,
                           key_dim: int, value_dim: int, values_from_keys: bool,
-                          frequencies: Optional[torch.Tensor] = None, write_kv: bool = True) -> torch.Tensor:
+                          frequencies: Optional[torch.Tensor] = None, write_kv: bool = True,
+                          in_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Rows ``[q: heads x key_dim | k: kv_heads x key_dim | v: kv_heads x value_dim]`` (no v columns with
         ``values_from_keys``: the values are the key columns as they come).  q and k are RMS-normed over their whole
         width (fp32 weights a column, or None) and rotated by ``rope_table`` (fp32 ``[positions, rotary_dim / 2,
         2]``, pairs of neighbours with ``interleaved``, else halves); q is returned as ``[T, heads x key_dim]``, k and v
         go to the rows' slots of ``cache [pages, page_size, kv_heads (key_dim + value_dim)]``.  ``frequencies`` (fp32
         ``[rotary_dim / 2]``) in the table's place: the angles ``position * f_i`` are formed in 32-bit in the kernel.
-        ``write_kv`` False: the rows hold q alone and nothing goes to the cache."""
+        ``write_kv`` False: the rows hold q alone and nothing goes to the cache.  ``in_bias`` (fp32, one number a column of
+        q, k and v): added first."""
         rows = src.shape[0]
+        assert in_bias is None or (in_bias.dtype == torch.float32 and in_bias.is_contiguous())
         num_pages, page_size, width = cache.shape
         assert src.stride(1) == 1 and cache.dtype == src.dtype and width == kv_heads * (key_dim + value_dim)
         assert src.shape[1] >= heads * key_dim + (0 if not write_kv else
@@ -1138,8 +1247,8 @@ class CudaOps:
         q = torch.empty(rows, heads * key_dim, dtype=src.dtype, device=src.device)
         rot = rotary_dim if (rope_table is not None or frequencies is not None) else 0
         assert frequencies is None or 2 * frequencies.shape[0] == rot
-        rc = self.lib.pih_window_qk_prepare(_DT[src.dtype], _ptr(src), c_ll(src.stride(0)), _ptr(q), _ptr(q_norm),
-                                            _ptr(k_norm), c_float(eps), _ptr(rope_table), _ptr(frequencies), rot,
+        rc = self.lib.pih_window_qk_prepare(_DT[src.dtype], _ptr(src), c_ll(src.stride(0)), _ptr(in_bias), _ptr(q),
+                                            _ptr(q_norm), _ptr(k_norm), c_float(eps), _ptr(rope_table), _ptr(frequencies), rot,
                                             1 if interleaved else 0,
                                             rope_table.shape[0] if rope_table is not None else 0, _ptr(positions),
                                             _ptr(slot_mapping), _ptr(cache), page_size, num_pages, rows, heads, kv_heads,
@@ -1152,12 +1261,12 @@ class CudaOps:
                          window: int, keep_first: int, softcap: float, bias: Optional[torch.Tensor],
                          sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], heads: int, kv_heads: int,
                          key_dim: int, value_dim: int, chunk: int = 0, scale_out: float = 1.0,
-                         out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         out: Optional[torch.Tensor] = None, gate_per: str = "head") -> torch.Tensor:
         """Attention of the step's rows (q prepared, ``[T, heads x key_dim]``) over the keys of their window (0: all), of
         their chunk of ``chunk`` places (0: all; chunks count from place 0 of the sequence) and the kept first keys, into
         ``out`` (a view) or a new tensor, times ``scale_out``; ``bias`` fp32 ``[heads, distances]`` by distance (the last column for every larger one),
         ``softcap`` 0: none, ``sink`` fp32 ``[heads]`` or None, ``gate`` ``[T, >= heads]`` (a view: column h is head
-        h's logit) or None.  Returns ``[T, heads x value_dim]``.
+        h's logit; with ``gate_per`` "column" ``[T, >= heads x value_dim]``, one logit a column) or None.  Returns ``[T, heads x value_dim]``.
 
         32-bit: a warp a (row, head) over the row's keys in a fixed order (the result does not depend on the step's
         make-up).  bf16: requests of more than 16 rows on the tensor-core kernel when it has an instance for the
@@ -1165,6 +1274,7 @@ class CudaOps:
         rows = q.shape[0]
         num_pages, page_size = cache.shape[0], cache.shape[1]
         assert q.is_contiguous() and cache.dtype == q.dtype and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1))
+        assert gate is None or gate.shape[1] >= heads * (value_dim if gate_per == "column" else 1)
         if out is None:
             out = torch.empty(rows, heads * value_dim, dtype=q.dtype, device=q.device)
         assert out.shape == (rows, heads * value_dim) and out.stride(1) == 1 and out.dtype == q.dtype
@@ -1198,7 +1308,8 @@ class CudaOps:
             _ptr(step.request_of_row), _ptr(step.positions), _ptr(step.cu_q), _ptr(getattr(step, "q_start", None)), rows,
             step.num_requests, heads, kv_heads, key_dim, value_dim, page_size, num_pages, c_float(scale),
             c_float(softcap or 0.0), _ptr(bias), distances, int(window), int(chunk), int(keep_first), _ptr(sink), _ptr(gate),
-            c_ll(gate.stride(0) if gate is not None else 0), tile, small, splits, _ptr(partial), self._err(), self._stream())
+            c_ll(gate.stride(0) if gate is not None else 0), 1 if gate_per == "column" else 0, tile, small, splits,
+            _ptr(partial), self._err(), self._stream())
         self._check(rc, "window_attention")
         self.launches += tile + (1 if splits > 1 else 0) + small - 1
         return out
@@ -1284,6 +1395,13 @@ class CudaOps:
                 self._check(rc, "gemm_skinny_bias_gelu")
                 return out
         return self.activation(self.linear(x, w), "gelu_erf", bias)
+
+    def softcap_(self, x: torch.Tensor, cap: float) -> torch.Tensor:
+        """``x = cap * tanh(x / cap)`` in place; x fp32, contiguous."""
+        assert x.dtype == torch.float32 and x.is_contiguous()
+        rc = self.lib.pih_softcap_rows(_ptr(x), c_ll(x.numel()), c_float(cap), self._stream())
+        self._check(rc, "softcap_rows")
+        return x
 
     def scale_(self, x: torch.Tensor, scale: float) -> torch.Tensor:
         """``x *= scale`` in place; x fp32, contiguous."""

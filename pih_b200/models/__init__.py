@@ -148,6 +148,8 @@ class CausalLM:
         logits = ops.linear(xn, self.head, out_dtype=torch.float32)
         if self.spec.logit_scale != 1.0:
             ops.scale_(logits, self.spec.logit_scale)
+        if self.spec.logit_softcap is not None:
+            ops.softcap_(logits, self.spec.logit_softcap)
         return logits
 
 

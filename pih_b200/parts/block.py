@@ -114,8 +114,8 @@ class OutNormBlock:
             return held[1]
         return self.rt.ops.stream_cast(h, self.rt.dtype)
 
-    def _add(self, h, y, norm, step, bias=None):
-        ops = self.rt.ops
+    def _add(self, h, y, norm, step, part):
+        ops, bias = self.rt.ops, getattr(part, "output_bias", None)
         x = ops.stream_norm_add(h, y, norm.weight_f32, norm.spec.eps, bias=bias,
                                 copy_dtype=self.rt.dtype if h.dtype != self.rt.dtype else None)
         step.stream_copy = (h, x) if x is not None else None
@@ -123,11 +123,61 @@ class OutNormBlock:
     def forward(self, h, delta, step, cache):
         if delta is not None:
             raise ValueError("a block with norms on its outputs takes a stream with nothing left to add")
-        self._add(h, self.mixer.forward(self._input(h, step), step, cache), self.norm_in, step)
+        self._add(h, self.mixer.forward(self._input(h, step), step, cache), self.norm_in, step, self.mixer)
         if self.ffn is not None:
             y = self.ffn.forward(self._input(h, step))
-            self._add(h, y, self.norm_post, step, bias=getattr(self.ffn, "output_bias", None))
+            self._add(h, y, self.norm_post, step, self.ffn)
         return h, None
+
+
+@register_block("sandwich")
+class SandwichBlock:
+    """``h += s1 * norm_in_out(mixer(norm_in(h))); h += s2 * norm_post_out(ffn(norm_post(h)))`` on a 32-bit stream: a norm
+    before and a norm behind each sub-layer, and (``spec.layer_scale``) a vector that multiplies the normed output.  The
+    vector goes into the weight of the norm behind (once, in 32-bit); that norm, the sum and the norm in front of the next
+    sub-layer are one kernel pass over a row (``Pending.norm``)."""
+
+    @classmethod
+    def expected_tensors(cls, spec):
+        out = PreNormBlock.expected_tensors.__func__(cls, spec)
+        for norm, role, scale in ((spec.norm_in_out, "norm_in_out", "scale_in"), (spec.norm_post_out, "norm_post_out", "scale_post")):
+            if norm is None:
+                continue
+            for rel, info in part_class("norm", norm.kind).expected_tensors(norm).items():
+                out[spec.names[role] + rel] = info
+            if spec.layer_scale:
+                out[spec.names[scale]] = TensorInfo((norm.width,), "one_plus_normal")
+        return out
+
+    def __init__(self, spec, weights, rt: Runtime):
+        PreNormBlock.__init__(self, spec, weights, rt)
+        if (spec.norm_post_out is None) != (spec.ffn is None) or spec.norm_in_out is None:
+            raise ValueError("a layer with norms before and behind its sub-layers names one of each a sub-layer")
+        self.behind = {}                    # (weight, eps) of the norm behind a sub-layer, the vector included
+        for sub, norm, role, scale in (("mixer", spec.norm_in_out, "norm_in_out", "scale_in"),
+                                       ("ffn", spec.norm_post_out, "norm_post_out", "scale_post")):
+            if norm is None:
+                continue
+            cls = part_class("norm", norm.kind)
+            part = cls(norm, _sub(weights, cls.expected_tensors(norm), spec.names[role]), rt)
+            if not hasattr(part, "weight_f32"):
+                raise TypeError("a norm behind a sub-layer needs a weight vector")
+            weight = part.weight_f32
+            if spec.layer_scale:
+                weight = weight * weights[spec.names[scale]].to(device=rt.device, dtype=torch.float32)
+            self.behind[sub] = (weight.contiguous(), float(norm.eps))
+
+    def forward(self, h, delta, step, cache):
+        x = self.norm_in.add_forward(h, delta)
+        if hasattr(self.mixer, "forward_pair") and self.mixer.pairs:
+            y, bias, pair = self.mixer.forward_pair(x, step, cache)
+        else:
+            y, bias, pair = self.mixer.forward(x, step, cache), getattr(self.mixer, "output_bias", None), None
+        delta = Pending(y, bias=bias, norm=self.behind["mixer"], pair=pair)
+        if self.ffn is not None:
+            y = self.ffn.forward(self.norm_post.add_forward(h, delta))
+            delta = Pending(y, bias=getattr(self.ffn, "output_bias", None), norm=self.behind["ffn"])
+        return h, delta
 
 
 @register_block("hyper")
@@ -159,6 +209,8 @@ class HyperBlock:
         for norm in (self.norm_in, self.norm_post):
             if norm is not None and not hasattr(norm, "weight_f32"):
                 raise TypeError("a layer over several streams norms with a weight vector")
+        if getattr(self.mixer, "output_bias", None) is not None:
+            raise TypeError("a layer over several streams takes no bias on its mixer's output")
         f32 = dict(device=rt.device, dtype=torch.float32)
         self.links = {}
         for sub in ("mixer", "ffn"):

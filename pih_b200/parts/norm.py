@@ -46,6 +46,9 @@ class RMSNorm:
         return self.add_forward(x, None, rows=rows)
 
     def add_forward(self, h, delta, rows=None):
+        if isinstance(delta, Pending) and delta.norm is not None:
+            return self.rt.ops.stream_norm_norm(h, delta.y, delta.norm[0], delta.norm[1], self.weight_f32, self.spec.eps,
+                                                bias=delta.bias, pair=delta.pair, rows=rows, out_dtype=self.rt.dtype)
         if isinstance(delta, Pending):
             return self.rt.ops.rmsnorm_stream(h, self.weight_f32, self.spec.eps, delta=delta.y, rows=rows,
                                               out_dtype=self.rt.dtype, scale=delta.scale, bias=delta.bias, again=delta.again,

@@ -30,6 +30,9 @@ mixer         ``cache_need() -> PagedKVNeed | PagedVectorNeed | StateNeed | Page
               from the first product's rows ``[T, n]`` (a view) to the second's
               ``[T, m]``, written into the view ``out`` and multiplied by
               ``scale``.  Such mixers can be run side by side (``parallel``).
+              ``output_bias`` (fp32 ``[hidden]``, optional): what is still to
+              be added to y.  A mixer whose output is a sum of two normed
+              products may hand them on (``forward_pair``; see ``Pending``).
 feed-forward  ``forward(x) -> y`` with x, y ``[T, hidden]``; ``output_bias``
               (fp32 ``[hidden]``, optional): what is still to be added to y.
 block         ``forward(h, delta, step, cache) -> (h, delta)``: the residual
@@ -89,12 +92,18 @@ class PagedStateNeed:
 class Pending:
     """What a 32-bit residual stream is still to receive, in this order: ``scale * (y + bias)``; ``factor * table[ids]``
     (``again`` = (table, ids, factor): the token's embedding once more); ``vector``.  The next norm adds it in its own
-    kernel.  Absent parts are None."""
+    kernel.  Absent parts are None.
+
+    ``norm`` = (weight, eps): the RMS norm of ``y + bias`` with that weight is what is added (then nothing else is).
+    ``pair`` = (y2, bias2, left weight, right weight, eps): the sum of ``y + bias`` and ``y2 + bias2``, each RMS-normed with
+    its weight, stands in the place of ``y + bias``; with ``norm`` only."""
     y: Optional[torch.Tensor] = None
     scale: float = 1.0
     bias: Optional[torch.Tensor] = None
     again: Optional[tuple] = None
     vector: Optional[torch.Tensor] = None
+    norm: Optional[tuple] = None
+    pair: Optional[tuple] = None
 
 
 @dataclass

@@ -50,7 +50,7 @@ class ComputedRotary:
     """The same rotate-half rotation without a table: the mixer's kernel forms ``angle = position * f_i`` in 32-bit
     from the frequencies ``f_i = theta^(-2i/rotary_dim)`` (computed in double here, rounded once) and takes its
     cosine and sine there.  No longest context has to be known.  ``interleaved``: the pairs are neighbours instead of
-    halves.  With ``stretch`` = (factor, low, high, original) the slow pairs are slowed down: with ``turns_i = original
+    halves.  ``slowdown`` divides every frequency.  With ``stretch`` = (factor, low, high, original) the slow pairs are slowed down: with ``turns_i = original
     f_i / (2 pi)`` and ``t_i = clamp((turns_i - low) / (high - low), 0, 1)`` the frequency is ``f_i (t_i + (1 - t_i) /
     factor)``."""
 
@@ -72,7 +72,10 @@ class ComputedRotary:
         import math
         pair = torch.arange(spec.rotary_dim // 2, dtype=torch.float64)
         f = torch.pow(torch.tensor(float(spec.theta), dtype=torch.float64), -2.0 * pair / spec.rotary_dim)
-        stretch = getattr(spec, "stretch", None)
+        slowdown, stretch = float(getattr(spec, "slowdown", 1.0)), getattr(spec, "stretch", None)
+        if slowdown <= 0:
+            raise ValueError("slowdown must be positive")
+        f = f / slowdown
         if stretch is None:
             return f
         factor, low, high, original = (float(v) for v in stretch)

@@ -3,7 +3,7 @@
 Router logits ``z = W_r x`` are 32-bit; ``s = softmax(z)`` over ALL ``experts + identity`` outputs.  The choice goes
 by ``s + correction``: outputs form ``groups`` equal groups of neighbours, a group's score is its largest choice
 score, only outputs of the ``groups_keep`` best groups can be chosen, and of those the ``top`` largest are (ties: the
-smaller index).  The weights are the chosen outputs' ``s`` (divided by their sum only with ``renormalize``).  Output
+smaller index).  The weights are the chosen outputs' ``s`` (divided by their sum only with ``renormalize``), times ``weight_scale``.  Output
 ``e < experts`` is the gated feed-forward ``W_down_e (silu(W_gate_e x) * (W_up_e x))``; an output behind them is an
 identity expert: the row itself.  A shared expert of the same form runs for every row and is added, multiplied by
 ``sigmoid(w_sg . x)``.
@@ -83,6 +83,7 @@ class ScoredMixtureOfExperts:
         out = ops.moe_experts(x, logits, self.w_gate_up, self.w_down, s.top,
                               routing=dict(outputs=s.outputs, correction=self.correction, groups=s.groups,
                                            groups_keep=s.groups_keep, renormalize=s.renormalize, scoring=self.scoring,
+                                           weight_scale=float(getattr(s, "weight_scale", 1.0)),
                                            gated=self.gated, weigh=self.weigh))
         if self.shared is not None:
             return ops.add_gated(out, self.shared.forward(x), logits[:, s.outputs] if self.shared_gate else None)

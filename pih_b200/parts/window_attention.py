@@ -6,13 +6,14 @@ reading key/value head ``h // (heads // kv_heads)``::
 
     s_j = scale q . k_j;   softcap: s_j <- c tanh(s_j / c);   bias: s_j <- s_j + rel[bucket(p - j), h]
     w_j = exp(s_j) / (sum over the seen keys of exp(s_i) + exp(sink_h))         (sink "zero": + 1; "none": no such term)
-    o   = sum_j w_j v_j;   head_gate: o <- o sigmoid(g_h),  g = W_g x
+    o   = sum_j w_j v_j;   head_gate: o <- o sigmoid(g_h),  g = W_g x;   column_gate: o <- o * sigmoid(W_g x), column by column
 
 What the spec switches on, each on its own (``WindowAttentionSpec``): short causal convolutions behind the q, k and v
 projections (the last ``taps - 1`` projected rows of a request are its state, in a state slot beside the pages); an
 RMS norm of q and of k over the WHOLE projection; values that are the keys as projected; a rotation of q and k; the
 bias by distance (the learned table ``[bias_rows, heads]`` is spread out once into one number a distance inside the
-window, so the kernels index it by the distance itself); capped scores; the gate a head.
+window, so the kernels index it by the distance itself); capped scores; the gate a head or a column; biases of the projections (those of q, k and v are added in 32-bit by the
+kernel that norms and rotates, that of the output travels on as ``output_bias``).
 
 The cache holds ONE vector per token, ``[k: kv_heads x key_dim | v: kv_heads x value_dim]`` after norm and rotation
 (``PagedVectorNeed`` with the window and the kept first tokens: the pages between them go back to the pool).  Scores,
@@ -80,6 +81,12 @@ class WindowAttention:
             out[n["sink"]] = TensorInfo((spec.heads,), "unit_normal")
         if spec.head_gate:
             out[n["gate"]] = TensorInfo((spec.heads, spec.hidden))
+        if spec.column_gate:
+            out[n["gate"]] = TensorInfo((spec.heads * spec.value_dim, spec.hidden))
+        if spec.biases:
+            for role in ("q", "k", "v", "o"):
+                if role + "_bias" in n and n[role] in out:
+                    out[n[role + "_bias"]] = TensorInfo((out[n[role]].shape[0],), "unit_normal")
         return out
 
     def __init__(self, spec, weights, rt: Runtime):
@@ -93,6 +100,8 @@ class WindowAttention:
             raise ValueError(f"sink must be 'learned', 'zero' or 'none', got {spec.sink!r}")
         if spec.bias_rows > 0 and (spec.bias_rows < 2 or spec.bias_far <= spec.bias_rows // 2):
             raise ValueError("a bias by distance needs at least 2 rows and a far distance beyond half of them")
+        if spec.head_gate and spec.column_gate:
+            raise ValueError("the gate is one number a head or one a column, not both")
         self.spec, self.rt = spec, rt
         self.own_kv = own = getattr(spec, "own_kv", True)
         n = spec.names
@@ -102,8 +111,15 @@ class WindowAttention:
         if own and not spec.values_from_keys:
             parts.append(weights[n["v"]])
         self.channels = sum(p.shape[0] for p in parts)
-        if spec.head_gate:
+        if spec.head_gate or spec.column_gate:
             parts.append(weights[n["gate"]])
+        self.in_bias = self.output_bias = None
+        if spec.biases:
+            roles = ["q"] + (["k"] if own else []) + (["v"] if own and not spec.values_from_keys else [])
+            self.in_bias = torch.cat([weights[n[r + "_bias"]].to(**f32) for r in roles]).contiguous()
+            self.output_bias = weights[n["o_bias"]].to(**f32).contiguous()
+            if spec.conv_taps > 0:
+                raise ValueError("biases in front of a short convolution are not supported")
         self.w_in = bind_matrix(torch.cat(parts, dim=0), rt)
         self.w_o = bind_matrix(weights[n["o"]], rt)
         self.w_conv = None
@@ -159,7 +175,7 @@ class WindowAttention:
         if cache.writable != self.own_kv:
             raise ValueError("window attention: the schedule entry's cache does not fit the mixer "
                              "(a mixer without keys and values reads another entry's cache, and only such a mixer)")
-        gate = proj[:, self.channels:] if s.head_gate else None
+        gate = proj[:, self.channels:] if s.head_gate or s.column_gate else None
         src = proj
         if self.w_conv is not None:
             state = cache.state if self._state_numbers() else proj.new_zeros((1, 1), dtype=torch.float32)
@@ -170,6 +186,8 @@ class WindowAttention:
             rotation = dict(frequencies=self.position.frequencies())
         if not self.own_kv:
             rotation["write_kv"] = False
+        if self.in_bias is not None:
+            rotation["in_bias"] = self.in_bias
         geometry = dict(heads=s.heads, kv_heads=s.kv_heads, key_dim=s.key_dim, value_dim=s.value_dim)
         q = ops.window_qk_prepare(src, q_norm=self.q_norm, k_norm=self.k_norm, eps=s.norm_eps or 0.0, rope_table=table,
                                   rotary_dim=self.position.rotary_dim if self.position is not None else 0,
@@ -178,4 +196,5 @@ class WindowAttention:
                                   **geometry, **rotation)
         return ops.window_attention(q, cache=cache.kv, block_table=cache.block_table, step=step, scale=s.scale,
                                     window=s.window, keep_first=s.keep_first, softcap=s.softcap or 0.0, bias=self.bias,
-                                    sink=self.sink, gate=gate, chunk=s.chunk, scale_out=scale, out=out, **geometry)
+                                    sink=self.sink, gate=gate, chunk=s.chunk, scale_out=scale, out=out,
+                                    gate_per="column" if s.column_gate else "head", **geometry)

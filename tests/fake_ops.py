@@ -173,6 +173,20 @@ class FakeOps:
             h.copy_(v)
         return (v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * weight).to(out_dtype)
 
+    def stream_norm_norm(self, h, y, add_weight, add_eps, weight, eps, bias=None, pair=None, rows=None, out_dtype=torch.bfloat16):
+        assert h.dtype == torch.float32
+        rms = lambda v, e: v / torch.sqrt((v * v).mean(-1, keepdim=True) + e)
+        u = y.float() + (bias if bias is not None else 0.0)
+        if pair is not None:
+            y2, bias2, left, right, pair_eps = pair
+            u = rms(u, pair_eps) * left + rms(y2.float() + (bias2 if bias2 is not None else 0.0), pair_eps) * right
+        v = h + rms(u, add_eps) * add_weight
+        if rows is not None:
+            v = v[rows.long()]
+        else:
+            h.copy_(v)
+        return (rms(v, eps) * weight).to(out_dtype)
+
     def linear_batched(self, x, w, out_dtype=None, rotate=None, gate=None):
         if rotate is not None:
             x = self.rotate_heads(x, **rotate)
@@ -232,8 +246,11 @@ class FakeOps:
                     out[t, h] = S[h].T @ qq
         return out
 
-    def gated_rmsnorm(self, o, gate, weight, eps, activation="silu", scale=1.0, out=None):
+    def gated_rmsnorm(self, o, gate, weight, eps, activation="silu", scale=1.0, out=None, divisor=None):
         T, heads, vdim = o.shape
+        weight = weight.view(-1, vdim)
+        if divisor is not None:
+            o = o / divisor[:, :, None]
         g = gate.float().view(T, heads, vdim)
         act = g * torch.sigmoid(g) if activation == "silu" else torch.sigmoid(g)
         y = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * weight * act * scale
@@ -241,6 +258,65 @@ class FakeOps:
         if out is None:
             return y.to(gate.dtype)
         return out.copy_(y)
+
+    def gated_part_rmsnorm(self, y, gate, weight, parts, eps, scale=1.0, out=None):
+        g = gate.float()
+        v = (y * g * torch.sigmoid(g)).view(y.shape[0], parts, -1)
+        v = (v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)).reshape(y.shape) * weight * scale
+        return v.to(gate.dtype) if out is None else out.copy_(v)
+
+    def memory_copies(self, value_dim):
+        return 2
+
+    def gated_linear(self, q, k, v, z, *, bias, temperature, q_scale, state, step, heads, key_dim, value_dim):
+        T = q.shape[0]
+        q, k = q.float().view(T, heads, key_dim), k.float().view(T, heads, key_dim)
+        v = v.float().view(T, heads, value_dim)
+        a = torch.exp(torch.nn.functional.logsigmoid(z + bias) / temperature).view(T, heads, key_dim)
+        out = torch.zeros(T, heads, value_dim)
+        for lo, hi, slot in self._requests(step):
+            S = state[slot, :heads * key_dim * value_dim].view(heads, key_dim, value_dim)
+            for t in range(lo, hi):
+                S.copy_(a[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :])
+                out[t] = torch.einsum("hdv,hd->hv", S, q[t]) * q_scale
+        return out
+
+    def state_space(self, C, B, x, dt, *, dt_bias, A, D, state, step, heads, groups, state_dim, value_dim):
+        T = x.shape[0]
+        per = heads // groups
+        C = C.float().view(T, groups, state_dim).repeat_interleave(per, dim=1)
+        B = B.float().view(T, groups, state_dim).repeat_interleave(per, dim=1)
+        x = x.float().view(T, heads, value_dim)
+        dt = torch.nn.functional.softplus(dt.float() + dt_bias)
+        out = torch.zeros(T, heads, value_dim)
+        for lo, hi, slot in self._requests(step):
+            S = state[slot, :heads * state_dim * value_dim].view(heads, state_dim, value_dim)
+            for t in range(lo, hi):
+                S.copy_(torch.exp(A * dt[t])[:, None, None] * S + (dt[t][:, None] * B[t])[:, :, None] * x[t][:, None, :])
+                out[t] = torch.einsum("hdv,hd->hv", S, C[t]) + D[:, None] * x[t]
+        return out
+
+    def matrix_memory(self, q, k, v, write, keep, *, write_bias, keep_bias, cap, floor, q_scale, state, step, heads, key_dim,
+                      value_dim):
+        T = q.shape[0]
+        q, k = q.float().view(T, heads, key_dim) * q_scale, k.float().view(T, heads, key_dim)
+        v = v.float().view(T, heads, value_dim)
+        i = cap * torch.tanh((write.float() + write_bias) / cap)
+        f = torch.nn.functional.logsigmoid(cap * torch.tanh((keep.float() + keep_bias) / cap))
+        out, div = torch.zeros(T, heads, value_dim), torch.zeros(T, heads)
+        a, b = heads * key_dim * value_dim, heads * key_dim
+        for lo, hi, slot in self._requests(step):
+            S = state[slot, :a].view(heads, key_dim, value_dim)
+            n, m = state[slot, a:a + b].view(heads, key_dim), state[slot, a + b:a + b + 2 * heads].view(heads, 2)
+            for t in range(lo, hi):
+                top = torch.maximum(f[t] + m[:, 0], i[t])
+                g, w = torch.exp(f[t] + m[:, 0] - top), torch.exp(i[t] - top)
+                S.copy_(g[:, None, None] * S + (w[:, None] * k[t])[:, :, None] * v[t][:, None, :])
+                n.copy_(g[:, None] * n + w[:, None] * k[t])
+                m.copy_(top[:, None].expand(heads, 2))
+                out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+                div[t] = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-top)) + floor
+        return out, div
 
     def selective_scan(self, u, dt, bc, z, *, dt_bias, A, D, state, step, scale=1.0, out=None):
         T, inner = u.shape
@@ -349,7 +425,9 @@ class FakeOps:
             c = torch.where(kept.repeat_interleave(n // groups, dim=1), c, torch.full_like(c, float("-inf")))
         idx = torch.argsort(c, dim=-1, descending=True, stable=True)[:, :top]
         wt = torch.gather(s, 1, idx)
-        return idx, wt / wt.sum(-1, keepdim=True) if routing.get("renormalize") else wt
+        if routing.get("renormalize"):
+            wt = wt / (wt.sum(-1, keepdim=True) + 1e-20)
+        return idx, wt * routing.get("weight_scale", 1.0)
 
     def moe_experts(self, x, logits, w_gate_up, w_down, top, routing=None):
         if routing is not None and not routing.get("gated", True):
@@ -519,8 +597,11 @@ class FakeOps:
         return u.to(out_dtype or torch.float32)
 
     def window_qk_prepare(self, src, *, q_norm, k_norm, eps, rope_table, rotary_dim, interleaved, positions, slot_mapping,
-                          cache, heads, kv_heads, key_dim, value_dim, values_from_keys, frequencies=None, write_kv=True):
+                          cache, heads, kv_heads, key_dim, value_dim, values_from_keys, frequencies=None, write_kv=True,
+                          in_bias=None):
         T = src.shape[0]
+        if in_bias is not None:
+            src = src[:, :in_bias.shape[0]].float() + in_bias
         nq, nk, nv = heads * key_dim, kv_heads * key_dim, kv_heads * value_dim
 
         def prepared(x, w):
@@ -542,10 +623,10 @@ class FakeOps:
                 x[..., :rotary_dim] = self._turn(x[..., :rotary_dim].clone(), positions, frequencies, interleaved)
             return x.reshape(T, -1)
 
-        q = prepared(src[:, :nq], q_norm).to(src.dtype)
+        q = prepared(src[:, :nq], q_norm).to(cache.dtype)
         if not write_kv:
             return q
-        k = prepared(src[:, nq:nq + nk], k_norm).to(src.dtype)
+        k = prepared(src[:, nq:nq + nk], k_norm).to(cache.dtype)
         v = src[:, nq:nq + nk] if values_from_keys else src[:, nq + nk:nq + nk + nv]
         flat = cache.view(-1, cache.shape[-1])
         for t, slot in enumerate(slot_mapping.tolist()):
@@ -557,7 +638,7 @@ class FakeOps:
         return q
 
     def window_attention(self, q, *, cache, block_table, step, scale, window, keep_first, softcap, bias, sink, gate, heads,
-                         kv_heads, key_dim, value_dim, chunk=0, scale_out=1.0, out=None):
+                         kv_heads, key_dim, value_dim, chunk=0, scale_out=1.0, out=None, gate_per="head"):
         T = q.shape[0]
         page_size = cache.shape[1]
         nk = kv_heads * key_dim
@@ -594,7 +675,9 @@ class FakeOps:
                 e = torch.exp(s - m)
                 den = e.sum() + (torch.exp(sink[h] - m) if sink is not None else 0.0)
                 o = (e / den) @ V[:, g]
-                if gate is not None:
+                if gate is not None and gate_per == "column":
+                    o = o * torch.sigmoid(gate[t, h * value_dim:(h + 1) * value_dim].float())
+                elif gate is not None:
                     o = o * torch.sigmoid(gate[t, h].float())
                 out[t, h] = o * scale_out
         out = out.reshape(T, heads * value_dim).to(q.dtype)
@@ -642,3 +725,6 @@ class FakeOps:
 
     def scale_(self, x, scale):
         return x.mul_(scale)
+
+    def softcap_(self, x, cap):
+        return x.copy_(cap * torch.tanh(x / cap))
