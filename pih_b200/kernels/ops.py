@@ -118,6 +118,7 @@ class CudaOps:
         lib.pih_attention_scratch_floats.restype = c_ll
         lib.pih_top_logprobs_scratch_words.restype = c_ll
         lib.pih_moe_route_words.restype = c_ll
+        lib.pih_linear_memory_scratch.restype = c_ll
 
     def _native_supports(self, block) -> bool:
         from .native_block import NativeBlocks
@@ -818,14 +819,38 @@ class CudaOps:
         assert gate0.stride(1) == 1 and (gate1 is None or gate1.stride(1) == 1) and state.dtype == torch.float32
         assert bias0.dtype == torch.float32 and (bias1 is None or bias1.dtype == torch.float32)
         out = torch.empty(T, heads, value_dim, dtype=torch.float32, device=q.device)
+        rows_of = (_DT[q.dtype], gate_kind, _ptr(q), c_ll(q.stride(0)), _ptr(k), c_ll(k.stride(0)), _ptr(v), c_ll(v.stride(0)))
+        # bf16: requests of more than 16 rows go by chunks on the tensor cores, the others (and everything in 32-bit, in an
+        # order of additions fixed by the row) token by token
+        scratch, small = None, 1
+        if q.dtype == torch.bfloat16 and self.chunked_memory:
+            big, small_rows, _ = self._row_plan(step)
+            need = self.lib.pih_linear_memory_scratch(*rows_of, T, step.num_requests, heads, key_dim, value_dim) if big else 0
+            if need > 0:
+                scratch = torch.empty(int(need), dtype=torch.float32, device=q.device)
+                small = 1 if small_rows > 0 else 0
+                self.launches += 3 + small
         rc = self.lib.pih_linear_memory(
-            _DT[q.dtype], gate_kind, _ptr(q), c_ll(q.stride(0)), _ptr(k), c_ll(k.stride(0)), _ptr(v), c_ll(v.stride(0)),
+            *rows_of,
             _ptr(gate0), c_ll(gate0.stride(0)), _ptr(gate1), c_ll(gate1.stride(0) if gate1 is not None else 0), _ptr(bias0),
             _ptr(bias1), _ptr(A), c_float(constant), c_float(floor), c_float(q_scale), _ptr(skip), _ptr(out), _ptr(divisor),
             _ptr(state), c_ll(state.stride(0)), _ptr(step.cu_q), _ptr(step.state_slots), T, step.num_requests, heads, groups,
-            key_dim, value_dim, self._stream())
+            key_dim, value_dim, _ptr(scratch), small, self._stream())
         self._check(rc, what)
         return out
+
+    chunked_memory = True                  # False: bf16 steps update the state token by token too
+
+    def _row_plan(self, step):
+        """``attention_plan`` of a step for one head a row group: (rows of the largest request of more than 16 rows, of the
+        largest other one, its context), worked out once a step."""
+        plans = getattr(step, "attention_plans", None)
+        plan = plans[1] if plans is not None and 1 in plans else None
+        if plan is None:
+            plan = self.attention_plan(step.host_cu_q, step.host_q_start, 1)
+            if plans is not None:
+                plans[1] = plan
+        return plan
 
     def gated_linear(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, *, bias: torch.Tensor,
                      temperature: float, q_scale: float, state: torch.Tensor, step, heads: int, key_dim: int,
