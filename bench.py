@@ -415,6 +415,25 @@ def _kedavik_config(width: int, layers: int, kinds=("mamba1", "parallel"), mlp: 
     return out
 
 
+def _bipulorn_config(width: int, layers: int, kinds=("gla", "parallel", "mlstm", "parallel"), moe: bool = True,
+                     window: int = 1024, vocab: int = 32768):
+    """Layer sizes that resemble a real model's at this width: a 128 x 128 matrix state a head and as many heads as
+    Tuganex's retention for the two plain recurrences (decays through 16 numbers); beside each other as many 128-wide
+    attention heads as Kedavik's (half as many key/value heads, half of each head rotated, windows of ``window`` keys) and a
+    state-space dual layer of twice the width (64-wide heads, 128 states, one group); Tuganex's experts (sixteen and two
+    identity experts, two chosen, a shared one)."""
+    heads = width // 128
+    mixers = {"gla": {"heads": heads, "dim": 128, "vdim": 128, "tau": 16.0, "decay_rank": 16},
+              "mlstm": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0},
+              "parallel": {"left": {"heads": heads, "kv_heads": max(1, heads // 2), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                    "rot": {"dims": 64, "base": 1e6, "scaling": {"factor": 4.0}}, "mask": {"size": window}},
+                           "right": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "norm_groups": 1, "conv": 4}}}
+    mlp = {"kind": "moe", "router": {"experts": 16, "identity": 2, "top": 2, "scale": 2.0}, "expert": {"ff": 3 * width // 2},
+           "shared": {"ff": width // 2}} if moe else None
+    return {"architecture": "Bipulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]], "mlp": mlp} for i in range(layers)]}
+
+
 def _dense_config(width: int, layers: int, vocab: int = 32768):
     return dict(QWEN3_0_6B, hidden_size=width, intermediate_size=3 * width, num_hidden_layers=layers,
                 num_attention_heads=width // 128 * 2, num_key_value_heads=width // 128, head_dim=128, vocab_size=vocab,
@@ -500,11 +519,117 @@ def _graph_us(fn, sets, calls: int = 24, repeats: int = 5) -> float:
     return sorted(times)[len(times) // 2]
 
 
+def _step_for_kernels(decode: bool, batch: int, prompt: int, context: int):
+    """(what the kernels want to know of a step, its rows, its requests): one prompt, or a decoded token of each of
+    ``batch`` requests behind ``context - 1`` others."""
+    import types
+    import torch
+    counts = [1] * batch if decode else [prompt]
+    starts = [context - 1] * batch if decode else [0]
+    cu = [0]
+    for c in counts:
+        cu.append(cu[-1] + c)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda:0")
+    return types.SimpleNamespace(
+        num_requests=len(counts), cu_q=i32(cu), q_start=i32(starts), state_slots=i32(range(len(counts))),
+        host_cu_q=cu, host_q_start=starts, attention_plans={}, meta=None,
+        request_of_row=i32([r for r, c in enumerate(counts) for _ in range(c)]),
+        positions=i32([starts[r] + i for r, c in enumerate(counts) for i in range(c)])), cu[-1], len(counts)
+
+
+def _bipulorn_kernels(width: int, batch: int, prompt: int, context: int):
+    """The kernels of the Bipulorn design beside the like kernel of another design, as ``_kedavik_kernels``."""
+    import torch
+    from pih_b200.kernels import get_ops
+    ops = get_ops(torch.device("cuda:0"))
+    hbm = peaks()[0]
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    H, d, inner, N = width // 128, 128, 2 * width, 128
+    rows_out = []
+    for decode in (False, True):
+        step, T, R = _step_for_kernels(decode, batch, prompt, context)
+        sets = 24 if decode else 6
+        rnd = lambda *shape, dtype=bf: [torch.randn(*shape, device=dev, dtype=dtype) for _ in range(sets)]
+        vec = lambda n: torch.randn(n, device=dev)
+
+        def add(name, us, nbytes):
+            rows_out.append({"kernel": name, "width": width, "step": f"decode x{batch}" if decode else f"prompt {prompt}",
+                             "us": round(us, 2), "MB": round(nbytes / 1e6, 2),
+                             "of_copy_peak": round(nbytes / (us * 1e-6) / (hbm * 1e9), 4)})
+
+        # the recurrences: q, k, v in, the read-outs out, the states in and out
+        qkv, gates, z = rnd(T, 3 * H * d), rnd(T, 2 * H), rnd(T, H * d, dtype=f32)
+        moved = T * H * d * (6 + 4) + 2 * R * H * d * d * 4
+        cut = lambda i: (qkv[i][:, :H * d], qkv[i][:, H * d:2 * H * d], qkv[i][:, 2 * H * d:])
+        kw = dict(step=step, heads=H, key_dim=d, value_dim=d)
+        st = rnd(R, H * d * d, dtype=f32)
+        bias, dm1 = vec(H * d), -torch.rand(H, device=dev) * 0.03
+        for chunked in (True, False) if not decode else (True,):
+            ops.chunked_memory = chunked
+            how = "" if chunked else ", token by token"
+            add("gated_linear" + how, _graph_us(lambda i: ops.gated_linear(*cut(i), z[i], bias=bias, temperature=16.0,
+                                                                          q_scale=d ** -0.5, state=st[i], **kw), sets), moved + T * H * d * 4)
+            sm = rnd(R, H * (d * d + d + ops.memory_copies(d)), dtype=f32)
+            b = vec(H)
+            add("matrix_memory" + how, _graph_us(lambda i: ops.matrix_memory(
+                *cut(i), gates[i][:, :H], gates[i][:, H:], write_bias=b, keep_bias=b, cap=15.0, floor=1e-6, q_scale=d ** -0.5,
+                state=sm[i], **kw), sets), moved + T * H * 8)
+            heads = inner // 64
+            xbc, dt, ss = rnd(T, inner + 2 * N), rnd(T, heads), rnd(R, heads * N * 64, dtype=f32)
+            A, bh = -torch.rand(heads, device=dev), vec(heads)
+            add("state_space" + how, _graph_us(lambda i: ops.state_space(
+                xbc[i][:, inner + N:], xbc[i][:, inner:inner + N], xbc[i][:, :inner], dt[i], dt_bias=bh, A=A, D=bh, state=ss[i],
+                step=step, heads=heads, groups=1, state_dim=N, value_dim=64), sets),
+                T * (inner * (2 + 4) + 4 * N + 2 * heads) + 2 * R * heads * N * 64 * 4)
+            del sm, xbc, dt, ss
+        ops.chunked_memory = True
+        add("retention (Tuganex)", _graph_us(lambda i: ops.retention(qkv[i][:, :2 * H * d], qkv[i][:, 2 * H * d:], frequencies=None,
+                                                                     decay_minus_one=dm1, key_scale=d ** -0.5, state=st[i], **kw), sets), moved)
+        del qkv, gates, z, st
+        # the attention with a gate a column beside the one with a gate a head, and what prepares its rows
+        G, pages, span = max(1, H // 2), -(-context // PAGE), 1024
+        tables = torch.arange(R * pages, dtype=torch.int32, device=dev).view(R, pages)
+        cache, src, gate = rnd(R * pages, PAGE, 2 * G * d), rnd(T, (H + 2 * G) * d), rnd(T, H * d)
+        geo = dict(heads=H, kv_heads=G, key_dim=d, value_dim=d)
+        common = dict(block_table=tables, step=step, scale=d ** -0.5, keep_first=0, softcap=0.0, bias=None, window=span, sink=None, **geo)
+        seen = R * span if decode else prompt
+        nbytes = T * H * d * 4 + seen * 2 * G * d * 2
+        q = [s_[:, :H * d].contiguous() for s_ in src]
+        add(f"window_attention, window of {span}, gate a column",
+            _graph_us(lambda i: ops.window_attention(q[i], cache=cache[i], gate=gate[i], gate_per="column", **common), sets), nbytes + T * H * d * 2)
+        add(f"window_attention, window of {span}, gate a head (Kedavik)",
+            _graph_us(lambda i: ops.window_attention(q[i], cache=cache[i], gate=gate[i], **common), sets), nbytes)
+        slots = (torch.arange(R, dtype=torch.int32, device=dev).repeat_interleave(T // R) * pages * PAGE
+                 + torch.arange(T, dtype=torch.int32, device=dev) % (T // R)).to(torch.int32)
+        freq, b_in = torch.rand(32, device=dev), vec((H + 2 * G) * d)
+        prep = dict(q_norm=None, k_norm=None, eps=0.0, rope_table=None, rotary_dim=64, positions=step.positions, slot_mapping=slots,
+                    values_from_keys=False, frequencies=freq, **geo)
+        for name, extra in (("window_qk_prepare, biases, neighbouring pairs", dict(interleaved=True, in_bias=b_in)),
+                            ("window_qk_prepare, halves (Kedavik)", dict(interleaved=False))):
+            add(name, _graph_us(lambda i: ops.window_qk_prepare(src[i], cache=cache[i], **prep, **extra), sets), T * (H + 2 * G) * d * 4)
+        del cache, src, gate, q
+        # the norms
+        y, gz, wv = rnd(T, inner, dtype=f32), rnd(T, inner), vec(inner)
+        add("gated_part_rmsnorm", _graph_us(lambda i: ops.gated_part_rmsnorm(y[i], gz[i], wv, 1, 1e-6), sets), T * inner * 8)
+        add("gated_rmsnorm (Rigotar)", _graph_us(lambda i: ops.gated_rmsnorm(y[i].view(T, -1, d), gz[i], wv[:d], 1e-6), sets), T * inner * 8)
+        del y, gz
+        h, a, b2 = rnd(T, width, dtype=f32), rnd(T, width), rnd(T, width)
+        w1 = vec(width)
+        add("stream_norm_norm", _graph_us(lambda i: ops.stream_norm_norm(h[i], a[i], w1, 1e-6, w1, 1e-6), sets), T * width * 12)
+        add("stream_norm_norm, a pair", _graph_us(lambda i: ops.stream_norm_norm(h[i], a[i], w1, 1e-6, w1, 1e-6, bias=w1,
+                                                                                pair=(b2[i], None, w1, w1, 1e-6)), sets), T * width * 14)
+        add("rmsnorm_stream (Rigotar)", _graph_us(lambda i: ops.rmsnorm_stream(h[i], w1, 1e-6, delta=a[i]), sets), T * width * 12)
+        add("stream_norm_add (Tuganex)", _graph_us(lambda i: ops.stream_norm_add(h[i], a[i], w1, 1e-6, copy_dtype=bf), sets), T * width * 12)
+        del h, a, b2
+        torch.cuda.empty_cache()
+    ops.check_errors()
+    return rows_out
+
+
 def _kedavik_kernels(width: int, batch: int, prompt: int, context: int):
     """The kernels of the Kedavik design beside the like kernel of another design, one prompt of ``prompt`` tokens and one
     decode step of ``batch`` requests: microseconds a call, the bytes that it has to move, and the fraction of the
     measured copy bandwidth that this makes.  Several sets of inputs and states in turn, together larger than L2."""
-    import types
     import torch
     from pih_b200.kernels import get_ops
     ops = get_ops(torch.device("cuda:0"))
@@ -513,21 +638,8 @@ def _kedavik_kernels(width: int, batch: int, prompt: int, context: int):
     heads, d, n, inner, group = width // 128, 128, 16, 2 * width, 2
     rows_out = []
 
-    def steps_of(decode):
-        counts = [1] * batch if decode else [prompt]
-        starts = [context - 1] * batch if decode else [0]
-        cu = [0]
-        for c in counts:
-            cu.append(cu[-1] + c)
-        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
-        return types.SimpleNamespace(
-            num_requests=len(counts), cu_q=i32(cu), q_start=i32(starts), state_slots=i32(range(len(counts))),
-            host_cu_q=cu, host_q_start=starts, attention_plans={}, meta=None,
-            request_of_row=i32([r for r, c in enumerate(counts) for _ in range(c)]),
-            positions=i32([starts[r] + i for r, c in enumerate(counts) for i in range(c)])), cu[-1], len(counts)
-
     for decode in (False, True):
-        step, T, R = steps_of(decode)
+        step, T, R = _step_for_kernels(decode, batch, prompt, context)
         sets = 24 if decode else 6
         rnd = lambda *shape, dtype=bf: [torch.randn(*shape, device=dev, dtype=dtype) for _ in range(sets)]
 
@@ -609,7 +721,19 @@ def design_run(args) -> int:
     batch, context, prompt, steps = args.batch, CONTEXT, PREFILL_TOKENS, max(8, args.steps // 4)
     with ClockSampler() as clocks:
         for width in (1024, 2048):
-            if args.design == "kedavik":
+            if args.design == "bipulorn":
+                # the design beside the models nearest to it (a matrix state with a fixed decay and the same experts; two mixers
+                # side by side) and the dense decoder; and each of its kinds of layer alone beside its like
+                cases = [("bipulorn", _bipulorn_config(width, 8)), ("tuganex", _tuganex_config(width, 8, mlps=("moe",))),
+                         ("kedavik", _kedavik_config(width, 8)), ("dense", _dense_config(width, 8))]
+                if width == 1024:
+                    cases += [(f"bipulorn {k} x4, no feed-forward", _bipulorn_config(width, 4, kinds=(k,), moe=False))
+                              for k in ("gla", "mlstm", "parallel")]
+                    cases += [("tuganex retention x4, no feed-forward", _tuganex_config(width, 4, kinds=("retention",), mlps=None)),
+                              ("kedavik parallel x4, no feed-forward", _kedavik_config(width, 4, kinds=("parallel",), mlp=False)),
+                              ("bipulorn gla x4 with experts", _bipulorn_config(width, 4, kinds=("gla",))),
+                              ("tuganex retention x4 with experts", _tuganex_config(width, 4, kinds=("retention",), mlps=("moe",)))]
+            elif args.design == "kedavik":
                 # the design beside the model nearest to it (a diagonal recurrence, a delta rule, attention) and the dense
                 # decoder; and each of its kinds of layer alone beside its like
                 cases = [("kedavik", _kedavik_config(width, 8)), ("rigotar", _rigotar_config(width, 8)),
@@ -684,7 +808,8 @@ def design_run(args) -> int:
                 del model
                 gc.collect()
                 torch.cuda.empty_cache()
-        kernels = {"kernels": _kedavik_kernels(1024, batch, prompt, context)} if args.design == "kedavik" else {}
+        alone = {"kedavik": _kedavik_kernels, "bipulorn": _bipulorn_kernels}.get(args.design)
+        kernels = {"kernels": alone(1024, batch, prompt, context)} if alone is not None else {}
         clock_summary = clocks.summary()
     print(json.dumps({"metric": f"prompt and decode tok/s of the {args.design.capitalize()} design beside the framework's other models",
                       "dtype": "bf16",
@@ -713,7 +838,7 @@ def main() -> int:
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
-    ap.add_argument("--design", default=None, choices=["rigotar", "tuganex", "pegopel", "sagelorn", "kedavik"],
+    ap.add_argument("--design", default=None, choices=["rigotar", "tuganex", "pegopel", "sagelorn", "kedavik", "bipulorn"],
                     help="instead of the recorded workload: this design's prompt and decode throughput beside the dense decoder's")
     ap.add_argument("--plain-launches", action="store_true",
                     help="launch kernels fully serialised instead of with programmatic dependent launch")

@@ -110,12 +110,15 @@ moe_route_scored_kernel(const float* __restrict__ logits, long long ld, const fl
     sum += sc[e];
   }
   sum = warp_sum(sum);
-  const float inv = scoring == 1 ? 1.0f : 1.0f / sum;         // (a sigmoid score stands for itself)
+  // (a sigmoid score stands for itself; a row whose logits are all NaN — padding holds whatever lay in memory — scores 0, so
+  // that its choice is one of the outputs like any row's)
+  const float inv = scoring == 1 ? 1.0f : (sum > 0.0f && sum < INFINITY ? 1.0f / sum : 0.0f);
 #pragma unroll
   for (int e = 0; e < kPer; ++e) {
     const int i = lane + 32 * e;
     sc[e] *= inv;
     ch[e] = (e * 32 < experts && i < experts) ? sc[e] + (correction != nullptr ? correction[i] : 0.0f) : -INFINITY;
+    if (!(ch[e] == ch[e])) ch[e] = -INFINITY;                  // comparisons with NaN would let the lanes choose differently
   }
   if (groups > 1) {
     float* score = route_smem + warp * 2 * groups;               // a group's score, then whether it is kept

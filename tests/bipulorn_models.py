@@ -73,10 +73,10 @@ B2 = {"architecture": "Bipulorn", "vocab": 263, "width": 64, "norm": {"eps": 1e-
                  layer(gla(2, 72, 16, 1.0, 33), moe(4, 2, 72, identity=0, scale=1.0, shared=8))]}
 B3 = {"architecture": "Bipulorn", "vocab": 83, "width": 50, "norm": {"eps": 1e-5},
       "layers": [layer(gla(1, 10, 6, 3.0, 1), moe(1, 1, 14, identity=1, scale=0.5, shared=10)),
-                 layer(pair(att(3, 1, 10, 6, 0.4, window=3, rot=6, base=30.0), ssd(3, 6, 5, 3, 9, 3)), moe(2, 2, 22)),
+                 layer(pair(att(3, 1, 10, 6, 0.4, window=3, rot=6, base=30.0), ssd(3, 6, 5, 3, 3, 3)), moe(2, 2, 22)),
                  layer(mlstm(1, 6, 10, 4.0), moe(3, 1, 10, identity=2, scale=3.0, shared=18)),
                  layer(pair(att(2, 2, 6, 10, 0.3), ssd(1, 14, 3, 1, 2, 5))),
-                 layer(pair(att(1, 1, 2, 4, -0.7, window=1), ssd(2, 3, 1, 2, 3, 2)))]}
+                 layer(pair(att(1, 1, 2, 4, -0.7, window=1), ssd(2, 3, 1, 2, 2, 2)))]}
 CONFIGS = {"B1": B1, "B2": B2, "B3": B3}
 SIGMA = {"B1": 0.15, "B2": 0.15, "B3": 0.2}
 
@@ -146,7 +146,7 @@ def random_config(seed):
             vdim = rnd.choice([4, 6, 8, 16, 24, 40, 64])
             inner = groups * per * vdim
             right = ssd(groups * per, vdim, rnd.choice([1, 4, 8, 16, 20, 40, 72]), groups,
-                        rnd.choice([n for n in (1, 2, 3, 4, 6, 8) if inner % n == 0]), rnd.choice([1, 2, 4]))
+                        rnd.choice([n for n in (1, 2, 3, 4, 6, 8) if inner % n == 0 and inner >= 4 * n]), rnd.choice([1, 2, 4]))
             mixer = pair(left, right)
         experts, identity = rnd.choice([1, 3, 6, 9]), rnd.choice([None, 0, 2, 5])
         mlp = moe(experts, rnd.randint(1, experts + (identity or 0)), rnd.choice([8, 24, 50]), identity=identity,

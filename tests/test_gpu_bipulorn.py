@@ -50,13 +50,15 @@ def _check(got, truth, dtype, what, rounding=None):
     if dtype == "float32":
         assert float(err.max()) < 5e-5, f"{what}: error {float(err.max()):.3e} of the logits' spread at row {int(err.argmax())}"
         return
-    bound = 0.03
-    if rounding is not None and (float(err.median()) >= bound or int((err > 3 * bound).sum()) > len(err) // 10):
+    bound, allowed = 0.03, len(err) // 10
+    if rounding is not None and (float(err.median()) >= bound or int((err > 3 * bound).sum()) > allowed):
         plain_err = rounding()
-        bound = max(bound, 1.5 * float(plain_err.median()), float(plain_err.quantile(0.9)) / 2)
+        bound = max(bound, 1.5 * float(plain_err.median()))
+        allowed = max(allowed, 3 * int((plain_err > 3 * bound).sum()) // 2)
     over = int((err > 3 * bound).sum())
-    assert float(err.median()) < bound and over <= len(err) // 10, \
-        f"{what}: median {float(err.median()):.3e}, {over} of {len(err)} positions beyond {3 * bound:.3f}, worst {float(err.max()):.3e}"
+    assert float(err.median()) < bound and over <= allowed, \
+        f"{what}: median {float(err.median()):.3e}, {over} of {len(err)} positions beyond {3 * bound:.3f} (at most {allowed}), " \
+        f"worst {float(err.max()):.3e}"
 
 
 def _rounding(folder, steps, requests, **kw):
@@ -344,3 +346,390 @@ def test_the_running_maximum_starts_at_zero_and_lives_on():
             _close(got / o.abs().amax(-1, keepdim=True).clamp(min=1e-30), o / o.abs().amax(-1, keepdim=True).clamp(min=1e-30),
                    3e-5 if dtype == torch.float32 else 1e-3, f"{dtype} {cuts}")
             _close(state[0, :mem.numbers], S, 1e-5 if dtype == torch.float32 else 1e-4)
+
+
+# -- attention, norms, gates -----------------------------------------------------------------------------------------------
+def _plain_rows(q, K, V, positions, scale, window, gate, group):
+    """softmax(q k scale) v over the last ``window`` keys (0: all), times the gate of the column."""
+    out = torch.zeros(q.shape[0], q.shape[1], V.shape[-1], dtype=F64)
+    for t, p in enumerate(positions):
+        lo = max(0, p - window + 1) if window else 0
+        for h in range(q.shape[1]):
+            s = (K[lo:p + 1, h // group] @ q[t, h]) * scale
+            out[t, h] = torch.softmax(s, dim=0) @ V[lo:p + 1, h // group]
+    return out * torch.sigmoid(gate).view(out.shape)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows_of_step", [260, 17, 5, 1])
+@pytest.mark.parametrize("window, dim, vdim", [(64, 64, 64), (50, 64, 128), (7, 32, 40), (1, 16, 24), (150, 96, 48), (0, 64, 64),
+                                               (40, 72, 136), (33, 20, 6)])
+def test_keys_that_stand_out_at_the_windows_edges(dtype, rows_of_step, window, dim, vdim):
+    """A key that scores high wherever it is seen, at every place in turn where rows exist for which it is the last one
+    inside the window (head 0) or at a page border (head 1); a gate a column; a prompt of several row tiles (the tensor-core
+    kernel in bf16), short portions and single rows (the warp kernel, its keys cut into parts).  Windows one place longer or
+    shorter would give something else."""
+    ops = _ops()
+    heads, kv_heads, page, n = 4, 2, 16, 300
+    g = torch.Generator().manual_seed(window + dim)
+    V = torch.randn(n, kv_heads, vdim, generator=g, dtype=F64)
+    K = 0.05 * torch.randn(n, kv_heads, dim, generator=g, dtype=F64)
+    unit = torch.zeros(dim, dtype=F64)
+    unit[3] = 1.0
+    edge = n - 1 - (window - 1 if window else 250)                # the last row's oldest key
+    for j in {edge, edge - 1, edge - 3, 40, 41}:
+        K[max(j, 0), 0] += (5.0 + 0.5 * (j % 3)) * unit
+    K[page - 1::page, 1] += 4.0 * unit
+    K[::page, 1] += 4.0 * unit
+    first = n - rows_of_step
+    positions = list(range(first, n))
+    q = 0.05 * torch.randn(rows_of_step, heads, dim, generator=g, dtype=F64) + 3.0 * unit
+    gate = torch.randn(rows_of_step, heads * vdim, generator=g, dtype=F64)
+    qd, Kd, Vd, gd = (x.to(dtype).double() for x in (q, K, V, gate))
+    want = 0.6 * _plain_rows(qd, Kd, Vd, positions, 0.5, window, gd, heads // kv_heads)
+    pages = -(-n // page)
+    order = torch.randperm(pages + 3, generator=g)[:pages]
+    cache = torch.zeros(pages + 3, page, kv_heads * (dim + vdim), dtype=dtype, device=DEV)
+    flat = torch.cat([Kd.reshape(n, -1), Vd.reshape(n, -1)], dim=1).to(dtype).to(DEV)
+    for i in range(pages):
+        rows = flat[i * page:(i + 1) * page]
+        cache[order[i], :rows.shape[0]] = rows
+    table = order.to(torch.int32).clone()
+    if window:
+        table[:max(0, first - window + 1) // page] = -1            # pages behind the window were given back
+    out = torch.full((rows_of_step, heads * vdim + 6), 9.0, dtype=dtype, device=DEV)
+    wide_gate = torch.cat([torch.full((rows_of_step, 3), 50.0, dtype=F64), gd], dim=1).to(dtype).to(DEV)[:, 3:]
+    ops.window_attention(qd.to(dtype).reshape(rows_of_step, -1).contiguous().to(DEV), cache=cache,
+                         block_table=table.to(DEV).reshape(1, -1).contiguous(),
+                         step=_step(positions, [0] * rows_of_step, [0, rows_of_step]), scale=0.5, window=window, keep_first=0,
+                         softcap=0.0, bias=None, sink=None, gate=wide_gate, gate_per="column", heads=heads, kv_heads=kv_heads,
+                         key_dim=dim, value_dim=vdim, scale_out=0.6, out=out[:, 2:2 + heads * vdim])
+    ops.check_errors()
+    assert bool((out[:, :2] == 9.0).all()) and bool((out[:, -4:] == 9.0).all())
+    got = out[:, 2:2 + heads * vdim].double().cpu().reshape(rows_of_step, heads, vdim)
+    limit = 1e-5 if dtype == torch.float32 else 2e-2
+    assert float((got - want).abs().max()) < limit * float(want.abs().max())
+    if window > 1:
+        for other in (window + 1, window - 1):                     # the check would see a fault
+            moved = 0.6 * _plain_rows(qd[-1:], Kd, Vd, positions[-1:], 0.5, other, gd[-1:], heads // kv_heads)
+            assert float((moved - want[-1:]).abs().max()) > 0.05 * float(want[-1].abs().max())
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("dim, vdim, rot", [(64, 128, 32), (64, 64, 64), (16, 24, 8), (10, 6, 6), (12, 20, 2), (320, 24, 320), (64, 48, 0)])
+def test_biases_and_rotation_of_neighbouring_pairs(dtype, dim, vdim, rot):
+    """q, k and v with their biases added before the rotation, into the queries' buffer and the cache; far positions; pairs of
+    halves and of neighbours; rows of padding write nothing."""
+    ops = _ops()
+    heads, kv_heads, page, T = 4, 2, 8, 21
+    g = torch.Generator().manual_seed(dim + rot)
+    cols = heads * dim + kv_heads * (dim + vdim)
+    src = torch.randn(T, cols + 8, generator=g).to(dtype)
+    bias = torch.randn(cols, generator=g)
+    positions = [0, 1, 2, 100, 1023] + list(range(3000, 3000 + T - 5))
+    slots = torch.arange(T, dtype=torch.int32) + 3
+    slots[6] = -2
+    for interleaved in (True, False):
+        if rot:
+            freq = torch.tensor([5000.0 ** (-2.0 * i / rot) / 4.0 for i in range(rot // 2)], dtype=F64)
+        cache = torch.zeros(4, page, kv_heads * (dim + vdim), dtype=dtype, device=DEV)
+        q = ops.window_qk_prepare(src.to(DEV), q_norm=None, k_norm=None, eps=0.0, rope_table=None, rotary_dim=rot,
+                                  interleaved=interleaved, positions=torch.tensor(positions, dtype=torch.int32, device=DEV),
+                                  slot_mapping=slots.to(DEV), cache=cache, heads=heads, kv_heads=kv_heads, key_dim=dim,
+                                  value_dim=vdim, values_from_keys=False, frequencies=freq.float().to(DEV) if rot else None,
+                                  in_bias=bias.to(DEV))
+        ops.check_errors()
+        x = src[:, :cols].double() + bias.double()
+
+        def turned(v, n):
+            v = v.reshape(T, n, dim)
+            if not rot:
+                return v
+            if interleaved:
+                return plain.rotate(v, torch.tensor(positions), {"dims": rot, "base": 5000.0, "scaling": {"factor": 4.0}})
+            ang = torch.tensor(positions, dtype=F64)[:, None] * freq[None, :]
+            c, s = torch.cos(ang)[:, None], torch.sin(ang)[:, None]
+            a, b = v[..., :rot // 2], v[..., rot // 2:rot]
+            return torch.cat([a * c - b * s, b * c + a * s, v[..., rot:]], dim=-1)
+
+        tol = 2e-3 if dtype == torch.float32 else 3e-2             # (32-bit angles of positions in the thousands)
+        _close(q, turned(x[:, :heads * dim], heads).reshape(T, -1), tol, "q")
+        flat = cache.view(-1, cache.shape[-1]).double().cpu()
+        want = torch.cat([turned(x[:, heads * dim:heads * dim + kv_heads * dim], kv_heads).reshape(T, -1),
+                          x[:, heads * dim + kv_heads * dim:]], dim=1)
+        for t, s in enumerate(slots.tolist()):
+            if s >= 0:
+                _close(flat[s], want[t], tol, f"cache row {t}")
+        assert float(flat[9].abs().max()) == 0.0 and float(flat[:3].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("width", [6, 72, 1000, 1024, 2050, 3001, 8192, 16384])
+def test_the_norm_behind_the_sum_and_the_next_norm(width):
+    """h += norm(y + bias) * w1, then norm(h) * w2; with a pair of outputs in y's place; stored back, or for gathered rows
+    not stored; sizes in 16-byte pieces, odd ones, and ones that need every piece a thread can hold."""
+    ops = _ops()
+    g = torch.Generator().manual_seed(width)
+    rows = 7
+    vec = lambda: torch.randn(width, generator=g)
+    h0, y, y2 = (torch.randn(rows, width, generator=g) for _ in range(3))
+    h0[3] *= 1e-3
+    y[4] *= 50.0
+    bias, bias2, left, right, w1, w2 = (vec() for _ in range(6))
+    pick = torch.tensor([6, 0, 3], dtype=torch.int32)
+    for dtype in (torch.float32, torch.bfloat16):
+        a, b = y.to(dtype), y2.to(dtype)
+        for parts in ("", "b", "p", "bp", "bpq"):
+            u = a.double() + (bias.double() if "b" in parts else 0.0)
+            kw = dict(bias=bias.to(DEV)) if "b" in parts else {}
+            if "p" in parts:
+                kw["pair"] = (b.to(DEV), bias2.to(DEV) if "q" in parts else None, left.to(DEV), right.to(DEV), 1e-3)
+                other = b.double() + (bias2.double() if "q" in parts else 0.0)
+                u = plain.rms_unit(u, 1e-3) * left.double() + plain.rms_unit(other, 1e-3) * right.double()
+            want = h0.double() + plain.rms_unit(u, 1e-5) * w1.double()
+            normed = plain.rms_unit(want, 1e-4) * w2.double()
+            tol = 3e-5 if dtype == torch.float32 else 2e-2
+            h = h0.to(DEV)
+            out = ops.stream_norm_norm(h, a.to(DEV), w1.to(DEV), 1e-5, w2.to(DEV), 1e-4, out_dtype=dtype, **kw)
+            assert out.dtype == dtype
+            _close(h, want, 1e-5)
+            _close(out, normed, tol)
+            h = h0.to(DEV)
+            out = ops.stream_norm_norm(h, a.to(DEV), w1.to(DEV), 1e-5, w2.to(DEV), 1e-4, out_dtype=dtype, rows=pick.to(DEV), **kw)
+            assert torch.equal(h.cpu(), h0)
+            _close(out, normed[pick.long()], tol)
+    ops.check_errors()
+
+
+@pytest.mark.parametrize("width, parts", [(96, 4), (96, 1), (50, 5), (3, 3), (4096, 1), (6000, 2), (2048, 8)])
+def test_norms_of_the_read_outs(width, parts):
+    """The gate before a norm in parts; the norm of a head divided by a number first, with a weight a head and column; both
+    into strided views, scaled; the capped logits."""
+    ops = _ops()
+    g = torch.Generator().manual_seed(width)
+    rows = 9
+    y, gate, w = torch.randn(rows, width, generator=g), torch.randn(rows, width + 3, generator=g), torch.randn(width, generator=g)
+    div = torch.rand(rows, parts, generator=g) + 1e-4
+    for dtype in (torch.float32, torch.bfloat16):
+        gd = gate.to(dtype)
+        tol = 1e-5 if dtype == torch.float32 else 2e-2
+        z = gd[:, 3:].double()
+        for what in ("parts", "heads"):
+            out = torch.full((rows, width + 4), 3.0, dtype=dtype, device=DEV)
+            if what == "parts":
+                ops.gated_part_rmsnorm(y.to(DEV), gd.to(DEV)[:, 3:], w.to(DEV), parts, 1e-4, scale=1.7, out=out[:, 2:width + 2])
+                ref = 1.7 * plain.part_norm(y.double() * plain.silu(z), parts, 1e-4) * w.double()
+            else:
+                o = y.view(rows, parts, -1).contiguous()
+                ops.gated_rmsnorm(o.to(DEV), gd.to(DEV)[:, 3:], w.to(DEV), 1e-4, activation="sigmoid", scale=1.7,
+                                  out=out[:, 2:width + 2], divisor=div.to(DEV))
+                ref = 1.7 * plain.rms_unit(o.double() / div.double()[:, :, None], 1e-4).reshape(rows, width) * w.double() * torch.sigmoid(z)
+            _close(out[:, 2:width + 2], ref, tol, what)
+            assert bool((out[:, :2] == 3.0).all()) and bool((out[:, width + 2:] == 3.0).all())
+    x = torch.linspace(-90, 90, 1001, device=DEV)[None, :].contiguous()
+    want = 7.5 * torch.tanh(x.double() / 7.5)
+    assert float((ops.softcap_(x, 7.5).double() - want).abs().max()) < 2e-6
+    ops.check_errors()
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows", [1, 8, 50, 300])
+def test_routing_weights_are_divided_and_scaled(rows, dtype):
+    """Experts and identity experts whose weights are the chosen scores over their sum, scaled — through the kernels of few
+    rows, of the library's grouped products and of the 32-bit path; the correction moves the choice and not the weights."""
+    ops = _ops()
+    g = torch.Generator().manual_seed(rows)
+    hidden, ff, experts, identity, top = 48, 24, 5, 3, 3
+    x = torch.randn(rows, hidden, generator=g).to(dtype)
+    logits, correction = torch.randn(rows, experts + identity + 1, generator=g), torch.randn(experts + identity, generator=g) * 0.3
+    bad = rows - 1 if rows > 1 else None                              # a row of padding may hold anything
+    if bad is not None:
+        logits[bad] = float("nan")
+    w = {}
+    for e in range(experts):
+        for n, shape in (("gate", (ff, hidden)), ("up", (ff, hidden)), ("down", (hidden, ff))):
+            w[f"e{e}.{n}"] = (torch.randn(*shape, generator=g) * 0.2).to(dtype)
+    gu = torch.stack([torch.cat([w[f"e{e}.gate"], w[f"e{e}.up"]]) for e in range(experts)])
+    dn = torch.stack([w[f"e{e}.down"] for e in range(experts)])
+    out = ops.moe_experts(x.to(DEV), logits.to(DEV), gu.to(DEV), dn.to(DEV), top,
+                          routing=dict(outputs=experts + identity, correction=correction.to(DEV), renormalize=True, weight_scale=2.3))
+    ops.check_errors()
+    ref = torch.zeros(rows, hidden, dtype=F64)
+    wd = {n: t.double() for n, t in w.items()}
+    out = out.double().cpu()
+    for t in range(rows):
+        if t == bad:
+            out[t] = 0.0
+            continue
+        for e, weight in plain.route(logits[t, :-1].double(), correction.double(), top, 2.3):
+            ref[t] += weight * (plain.gated(x[t].double(), wd, f"e{e}.") if e < experts else x[t].double())
+    _close(out, ref, 1e-5 if dtype == torch.float32 else 2e-2)
+
+
+# -- whole models ------------------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("name", ["B1", "B2"])
+def test_batches_against_each_request_alone(dirs, name):
+    """Unequal requests side by side in one step — a long portion, a short one, single tokens — give each request
+    what it gets alone (32-bit: every reduction has an order fixed by the row)."""
+    from pih_b200.engine import StepEntry
+    from pih_b200.engine.factory import create_runner
+    requests = traces.make_requests(bm.CONFIGS[name]["vocab"], [61, 18, 40, 9], seed=8)
+    alone = {}
+    for rid, toks in requests.items():
+        _, _, _, runner = create_runner(dirs[name], "float32", page_size=16, max_cache_tokens=128, max_requests=1)
+        alone[rid] = traces.replay(runner, traces.whole({rid: toks}))[rid]
+    _, model, cache, runner = create_runner(dirs[name], "float32", page_size=16, max_cache_tokens=256, max_requests=4)
+    cuts = {"r0": [33, 27, 1], "r1": [1, 16, 1], "r2": [2, 37, 1], "r3": [7, 1, 1]}
+    got, at = {rid: [] for rid in requests}, {rid: 0 for rid in requests}
+    for i in range(3):
+        entries = []
+        for rid, toks in requests.items():
+            n = cuts[rid][i]
+            entries.append(StepEntry(rid, toks[at[rid]:at[rid] + n], list(range(n))))
+            at[rid] += n
+        logits = runner.step(entries)
+        j = 0
+        for e in entries:
+            got[e.rid].append(logits[j:j + len(e.tokens)].clone())
+            j += len(e.tokens)
+    model.rt.ops.check_errors()
+    for rid in requests:
+        assert float((torch.cat(got[rid]).cpu() - alone[rid]).abs().max()) < 1e-5 * float(alone[rid].abs().max()), rid
+
+
+@pytest.mark.parametrize("seed", range(12))
+def test_configurations_drawn_at_random(tmp_path, seed):
+    """Sizes, orders of layers and constants drawn at random (odd sizes and sizes that only the plain kernels take among
+    them): a mixed schedule in 32-bit against the plain implementation position by position, and in bfloat16 within
+    rounding."""
+    from pih_b200.engine.factory import create_runner
+    raw = bm.random_config(seed)
+    requests = traces.make_requests(raw["vocab"], [150, 45, 33, 18, 1, 2], seed=seed)
+    steps = traces.mixed(requests, seed=seed, max_live=3, max_portion=60)
+    d = bm.write_model(tmp_path / "m", raw, seed=seed, sigma=0.15)
+    kw = dict(page_size=16, max_cache_tokens=traces.peak_tokens(steps, round_to=16), max_requests=3)
+    for dtype in ("float32", "bfloat16"):
+        _, model, cache, runner = create_runner(d, dtype, **kw)
+        got = traces.replay(runner, steps)
+        model.rt.ops.check_errors()
+        _check(got, bm.plain_logits(d, requests), dtype, f"seed {seed} {dtype}", rounding=_rounding(d, steps, requests, **kw))
+        cache.check()
+
+
+def test_long_decoding(dirs):
+    """A short prompt and 300 tokens one by one: pages fill and go back behind the windows, the states run on."""
+    from pih_b200.engine.factory import create_runner
+    for name in ("B1", "B3"):
+        requests = traces.make_requests(bm.CONFIGS[name]["vocab"], [310], seed=9)
+        steps = traces.tail_decode(requests, tail=300)
+        _, model, cache, runner = create_runner(dirs[name], "float32", page_size=8, max_cache_tokens=320, max_requests=1)
+        _check(traces.replay(runner, steps), bm.plain_logits(dirs[name], requests), "float32", f"{name} long decoding")
+        model.rt.ops.check_errors()
+
+
+@pytest.mark.parametrize("cuda_graphs", [False, True])
+@pytest.mark.parametrize("name", ["B1", "B2", "B3"])
+def test_greedy_generation_through_the_engine(dirs, name, cuda_graphs):
+    """Engine.complete (scheduler, cache, sampler, graphs, padded steps, ids fed on the device) against greedy decoding
+    with the plain implementation; three requests at once with room for two, so they queue."""
+    from pih_b200.engine import Engine
+    cfg, w = bm.load_plain(dirs[name])
+    prompts = list(traces.make_requests(bm.CONFIGS[name]["vocab"], [9, 21, 5], seed=13).values())
+    new, want = 12, []
+    for p in prompts:
+        _, logits, state = plain.model_layers(cfg, w, p)
+        toks = [int(logits[-1].argmax())]
+        while len(toks) < new:
+            _, logits, state = plain.model_layers(cfg, w, toks[-1:], state)
+            toks.append(int(logits[-1].argmax()))
+        want.append(toks)
+    engine = Engine(dirs[name], "float32", page_size=16, max_cache_tokens=256, maximum_batch_sequences=2,
+                    maximum_batch_tokens=64, maximum_context_tokens=64, cuda_graphs=cuda_graphs)
+    results = engine.complete_batch(prompts, max_tokens=new, temperature=0.0, ignore_eos=True)
+    engine.rt.ops.check_errors()
+    for r, expect in zip(results, want):
+        assert r["token_ids"] == expect
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_graphs_and_padded_steps_against_plain_launches(dirs, dtype):
+    """The same mixed requests through a runner that pads its steps and replays them from graphs and through one that
+    does not: padding leaves states, pages and logits alone."""
+    from pih_b200.engine import StepEntry
+    from pih_b200.engine.factory import create_runner
+    requests = traces.make_requests(bm.B1["vocab"], [33, 20, 47], seed=17)
+    logits = []
+    for graphs in (False, True):
+        _, model, cache, runner = create_runner(dirs["B1"], dtype, page_size=16, max_cache_tokens=512, max_requests=4,
+                                                cuda_graphs=graphs)
+        out = []
+        for turn in range(3):                                        # the same shapes again: seen, captured, replayed
+            at = {r: 0 for r in requests}
+            for cuts in ([17, 3, 30], [1, 9, 1], [9, 1, 10], [1, 1, 1], [1, 1, 1], [4, 5, 4]):
+                entries = []
+                for rid, n in zip(requests, cuts):
+                    entries.append(StepEntry(f"{rid}.{turn}", requests[rid][at[rid]:at[rid] + n], [n - 1]))
+                    at[rid] += n
+                out.append(runner.step(entries).clone())
+            for rid in requests:
+                runner.finish(f"{rid}.{turn}")
+        model.rt.ops.check_errors()
+        logits.append(torch.stack([o.float() for o in out]))
+    scale = float(logits[0].std())
+    assert float((logits[0] - logits[1]).abs().max()) < (1e-5 if dtype == "float32" else 0.2) * scale
+    six = logits[1].view(3, 6, *logits[1].shape[1:])
+    assert float((six[0] - six[2]).abs().max()) < (1e-5 if dtype == "float32" else 0.2) * scale
+
+
+def test_command_lines(dirs, tmp_path):
+    """bin/pih-worker makes a random Bipulorn model from a configuration file and generates from it; bin/trace_run replays
+    a trace on it, in both precisions; all agree with the plain implementation."""
+    import json
+    import os
+    import subprocess
+    import sys
+
+    import numpy as np
+    from conftest import ROOT
+    worker = [sys.executable, os.path.join(ROOT, "bin", "pih-worker")]
+    cfg_file = tmp_path / "config.json"
+    cfg_file.write_text(json.dumps(bm.B1))
+    folder = str(tmp_path / "made")
+    proc = subprocess.run(worker + ["--random-model", folder, "--config", str(cfg_file), "--seed", "4", "--sigma", "0.15"],
+                          capture_output=True, text=True, timeout=600)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    prompt = [5, 17, 3, 200, 9]
+    proc = subprocess.run(worker + ["--model", folder, "--generate-tokens", ",".join(map(str, prompt)), "--max-tokens", "7",
+                                    "--dtype", "float32", "--ignore-eos"], capture_output=True, text=True, timeout=600)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    res = json.loads(proc.stdout.strip().splitlines()[-1])
+    cfg, w = bm.load_plain(folder)
+    toks = list(prompt)
+    for _ in range(7):
+        toks.append(int(plain.model_layers(cfg, w, toks)[1][-1].argmax()))
+    assert res["token_ids"] == toks[len(prompt):]
+
+    requests = traces.make_requests(bm.B1["vocab"], [40, 9, 23], seed=6)
+    steps = traces.mixed(requests, seed=1, max_live=3)
+    for s_ in steps:
+        for e in s_["entries"]:
+            e["want"] = e["want"][-1:]                              # the last place of every portion
+    truth = bm.plain_logits(folder, requests)
+    for dtype, tol in (("float32", 1e-4), ("bfloat16", 0.1)):
+        out_dir = str(tmp_path / dtype)
+        cmd = [sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", dtype, "--out", out_dir,
+               "--max-tokens", str(traces.peak_tokens(steps))]
+        proc = subprocess.run(cmd, input="\n".join(json.dumps(s_) for s_ in steps) + "\n", capture_output=True, text=True,
+                              timeout=600)
+        assert proc.returncode == 0, proc.stderr[-2000:]
+        assert [l for l in proc.stdout.splitlines() if l.startswith("done ")] == [f"done {s_['step']}" for s_ in steps]
+        at = {rid: 0 for rid in requests}
+        over = total = 0
+        for s_ in steps:
+            got = np.fromfile(os.path.join(out_dir, f"{s_['step']}.f32"), dtype="<f4").reshape(-1, bm.B1["vocab"])
+            for j, e in enumerate(s_["entries"]):
+                at[e["id"]] += len(e["tokens"])
+                ref = truth[e["id"]][at[e["id"]] - 1].numpy()
+                total += 1
+                over += int(np.abs(got[j] - ref).max() >= tol * max(1.0, np.abs(ref).max()))
+        # (in bfloat16 a rounded router logit may choose another expert at a few places)
+        assert over <= (0 if dtype == "float32" else total // 10), (dtype, over, total)
