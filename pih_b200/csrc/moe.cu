@@ -78,6 +78,7 @@ moe_route_kernel(const float* __restrict__ logits, int rows, int experts, int to
 // ``keep`` best of ``groups`` equal groups of neighbours (a group's score: its largest choice score; the others count
 // as minus infinity); the ``top`` largest are chosen (ties: the smaller index) and weigh with their s, divided by the
 // chosen ones' sum only with ``renormalize``, and times ``weight_scale``.  One warp a row; ``flags``: [warps][groups] ints of shared memory.
+template <int kPer>                                              // 32 kPer experts at most
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction, int rows,
                         int experts, int top, int groups, int keep, int renormalize, int scoring, float weight_scale,
@@ -90,7 +91,6 @@ moe_route_scored_kernel(const float* __restrict__ logits, long long ld, const fl
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (row >= rows) return;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  constexpr int kPer = 32;                                       // experts <= 1024
   float sc[kPer], ch[kPer];
   uint32_t taken = 0;
   float mx = -INFINITY;
@@ -559,7 +559,8 @@ extern "C" int pih_moe_route_scored(const void* logits, long long ld, const void
   int* row_of = pos_of + slots;
   int* counts = row_of + slots;
   int* plan = counts + experts;
-  launch_kernel(moe_route_scored_kernel, dim3((rows + 3) / 4), dim3(128), 4 * 2 * groups * sizeof(float), s,
+  auto kernel = experts <= 32 ? moe_route_scored_kernel<1> : (experts <= 128 ? moe_route_scored_kernel<4> : moe_route_scored_kernel<32>);
+  launch_kernel(kernel, dim3((rows + 3) / 4), dim3(128), 4 * 2 * groups * sizeof(float), s,
                 static_cast<const float*>(logits), ld, static_cast<const float*>(correction), rows, experts, top, groups,
                 keep, renormalize, scoring, weight_scale, expert_of, static_cast<float*>(weight_of), rank_of,
                 grouped ? counts : static_cast<int*>(nullptr), pos_of);

@@ -333,7 +333,8 @@ stream_norm_norm_kernel(float* __restrict__ h, const NormedOutput<TD> add, const
 // replaces it afterwards.
 constexpr int kConvRows = 128;
 
-template <typename T>
+// kTaps: the number of taps at most; an instance of the usual sizes shifts and multiplies no more than it has to.
+template <typename T, int kTaps>
 __global__ void __launch_bounds__(256)
 causal_conv_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const float* __restrict__ in_bias,
                    const float* __restrict__ out_bias, T* __restrict__ out, long long ldo, int channels, int taps,
@@ -349,9 +350,9 @@ causal_conv_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__
   if (n <= t_first || slot < 0 || c >= channels) return;
   const int hist_n = taps - 1;
   const float* st = state + slot * state_stride + state_offset;       // [taps-1][channels]
-  float wr[kMaxTaps];
+  float wr[kTaps];
 #pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j) wr[j] = j < taps ? to_float<T>(w[static_cast<long long>(c) * taps + j]) : 0.0f;
+  for (int j = 0; j < kTaps; ++j) wr[j] = j < taps ? to_float<T>(w[static_cast<long long>(c) * taps + j]) : 0.0f;
   const float ib = in_bias != nullptr ? in_bias[c] : 0.0f;
   const float ob = out_bias != nullptr ? out_bias[c] : 0.0f;
   // a token lane takes a run of consecutive rows and keeps the last taps inputs in registers: every input is read once
@@ -362,22 +363,22 @@ causal_conv_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__
     return s >= 0 ? to_float<T>(x[static_cast<long long>(lo + s) * ldx + c]) + ib
                   : st[static_cast<long long>(hist_n + s) * channels + c];
   };
-  float held[kMaxTaps];                                       // held[j] = in(t - hist_n + j), j < taps
+  float held[kTaps];                                       // held[j] = in(t - hist_n + j), j < taps
 #pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j) held[j] = (j + 1 < taps) ? input(t0 - hist_n + j) : 0.0f;
+  for (int j = 0; j < kTaps; ++j) held[j] = (j + 1 < taps) ? input(t0 - hist_n + j) : 0.0f;
 #pragma unroll 4
   for (int t = t0; t < t1; ++t) {
     const float newest = input(t);
     float acc = 0.0f;
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j) {
+    for (int j = 0; j < kTaps; ++j) {
       if (j < taps) {
         const float v = j + 1 == taps ? newest : held[j];
         acc = fmaf(wr[j], v, acc);
       }
     }
 #pragma unroll
-    for (int j = 0; j + 1 < kMaxTaps; ++j) held[j] = j + 2 == taps ? newest : held[j + 1];
+    for (int j = 0; j + 1 < kTaps; ++j) held[j] = j + 2 == taps ? newest : held[j + 1];
     acc += ob;
     if (activation == 1) acc = acc / (1.0f + expf(-acc));
     out[static_cast<long long>(lo + t) * ldo + c] = from_float<T>(acc);
@@ -783,7 +784,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, l
 
 // Block (row, part): y fp32 [rows, width] times silu(gate [rows, ldg]), the part's own RMS norm, a weight a column.
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
 gated_part_rmsnorm_kernel(const float* __restrict__ y, const T* __restrict__ gate, long long ldg,
                           const float* __restrict__ weight, T* __restrict__ out, long long ldo, int width, int part,
                           float eps, float out_scale) {
@@ -1011,12 +1012,17 @@ extern "C" int pih_causal_conv(int dtype, const void* x, long long ldx, const vo
   dim3 grid(requests, (channels + 31) / 32, (rows + kConvRows - 1) / kConvRows), block(32, 8);
   dim3 grid_h(requests, (channels + 127) / 128);
   if (grid.y > 65535 || grid.z > 65535) return PIH_ERR_UNSUPPORTED;
+#define PIH_CONV_TAPS(T, N)                                                                                            \
+  launch_kernel(causal_conv_kernel<T, N>, grid, block, 0, s, static_cast<const T*>(x), ldx, static_cast<const T*>(w),  \
+                static_cast<const float*>(in_bias), static_cast<const float*>(out_bias), static_cast<T*>(out), ldo,    \
+                channels, taps, activation, static_cast<const float*>(state), state_stride, state_offset,              \
+                static_cast<const int*>(cu_q), static_cast<const int*>(state_slots))
 #define PIH_CONV(T)                                                                                                    \
   do {                                                                                                                 \
-    launch_kernel(causal_conv_kernel<T>, grid, block, 0, s, static_cast<const T*>(x), ldx, static_cast<const T*>(w),    \
-                  static_cast<const float*>(in_bias), static_cast<const float*>(out_bias), static_cast<T*>(out), ldo,  \
-                  channels, taps, activation, static_cast<const float*>(state), state_stride, state_offset,            \
-                  static_cast<const int*>(cu_q), static_cast<const int*>(state_slots));                                \
+    if (taps <= 2) PIH_CONV_TAPS(T, 2);                                                                                \
+    else if (taps == 3) PIH_CONV_TAPS(T, 3);                                                                           \
+    else if (taps == 4) PIH_CONV_TAPS(T, 4);                                                                           \
+    else PIH_CONV_TAPS(T, kMaxTaps);                                                                                   \
     PIH_LAUNCH_CHECK();                                                                                                \
     if (taps > 1)                                                                                                      \
       launch_kernel(causal_conv_history_kernel<T>, grid_h, dim3(128), 0, s, static_cast<const T*>(x), ldx,             \
@@ -1027,6 +1033,7 @@ extern "C" int pih_causal_conv(int dtype, const void* x, long long ldx, const vo
   else if (dtype == PIH_BF16) PIH_CONV(bf16);
   else return PIH_ERR_BAD_ARGUMENT;
 #undef PIH_CONV
+#undef PIH_CONV_TAPS
   PIH_LAUNCH_CHECK();
   return 0;
 }
@@ -1165,7 +1172,7 @@ extern "C" int pih_gated_part_rmsnorm(int dtype, const void* y, const void* gate
   if (parts > 65535) return PIH_ERR_UNSUPPORTED;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int part = width / parts;
-  const int threads = part >= 1024 ? 256 : (part >= 256 ? 128 : (part >= 64 ? 64 : 32));
+  const int threads = part >= 2048 ? 512 : (part >= 1024 ? 256 : (part >= 256 ? 128 : (part >= 64 ? 64 : 32)));
 #define PIH_GPN(T)                                                                                                     \
   launch_kernel(gated_part_rmsnorm_kernel<T>, dim3(rows, parts), dim3(threads), 0, s, static_cast<const float*>(y),      \
                 static_cast<const T*>(gate), ldg, static_cast<const float*>(weight), static_cast<T*>(out), ldo, width,  \

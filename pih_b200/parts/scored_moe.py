@@ -63,7 +63,10 @@ class ScoredMixtureOfExperts:
         self.spec, self.rt = spec, rt
         n = spec.names
         router = [weights[n["router"]]] + ([weights[n["shared_gate"]]] if self.shared_gate else [])
-        self.w_router = bind_matrix(torch.cat(router, dim=0), rt)          # the shared expert's gate is the last row
+        # the shared expert's gate is the row behind the outputs'; rows of zeros make a multiple of 8 (columns that nothing
+        # reads: a product whose rows begin at multiples of 16 bytes)
+        rows = sum(r.shape[0] for r in router)
+        self.w_router = bind_matrix(torch.cat(router + [router[0].new_zeros((-rows % 8, router[0].shape[1]))], dim=0), rt)
         self.correction = None
         if getattr(spec, "correction", True):
             self.correction = weights[n["correction"]].to(device=rt.device, dtype=torch.float32).contiguous()
@@ -79,7 +82,7 @@ class ScoredMixtureOfExperts:
 
     def forward(self, x):
         s, ops = self.spec, self.rt.ops
-        logits = ops.linear(x, self.w_router, out_dtype=torch.float32)      # [T, outputs (+ 1)], 32-bit
+        logits = ops.linear(x, self.w_router, out_dtype=torch.float32)      # [T, outputs (+ 1) (+ zeros)], 32-bit
         out = ops.moe_experts(x, logits, self.w_gate_up, self.w_down, s.top,
                               routing=dict(outputs=s.outputs, correction=self.correction, groups=s.groups,
                                            groups_keep=s.groups_keep, renormalize=s.renormalize, scoring=self.scoring,
