@@ -375,12 +375,19 @@ memory_channels_kernel(const MemoryArgs p) {
   float* L = p.log_decay + static_cast<long long>(c.first) * channels + at;
   const float bias = p.bias0[at];
   float sum = 0.0f;
-#pragma unroll 8
-  for (int t = 0; t < c.rows; ++t) {
-    // log sigmoid by the special-function unit: its error is far below a bf16 rounding of z's inputs
-    const float x = -(z[t * p.ld0] + bias);
-    sum -= (fmaxf(x, 0.0f) + __logf(1.0f + __expf(-fabsf(x)))) * p.constant;
-    L[static_cast<long long>(t) * channels] = sum;
+  constexpr int kAhead = 16;                                 // rows asked for together
+  for (int t0 = 0; t0 < c.rows; t0 += kAhead) {
+    float x[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) x[i] = t0 + i < c.rows ? z[(t0 + i) * p.ld0] : 0.0f;
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      if (t0 + i >= c.rows) continue;
+      // log sigmoid by the special-function unit: its error is far below a bf16 rounding of z's inputs
+      const float y = -(x[i] + bias);
+      sum -= (fmaxf(y, 0.0f) + __logf(1.0f + __expf(-fabsf(y)))) * p.constant;
+      L[static_cast<long long>(t0 + i) * channels] = sum;
+    }
   }
 }
 
@@ -436,37 +443,60 @@ memory_chunk_state_kernel(const MemoryArgs p) {
   const int channels = p.heads * p.dim;
   const long long last = c.first + c.rows - 1;
   const float end = GATE == kChannel ? 0.0f : p.log_decay[last * p.heads + h];
-  for (int e = threadIdx.x; e < kChunkRows * (kTileDim / 8); e += blockDim.x) {
-    const int row = e / (kTileDim / 8), col = (e % (kTileDim / 8)) * 8;
+  constexpr int kPieces = kChunkRows * (kTileDim / 8) / 128;   // of 8 keys a thread; all asked for before the first is used
+  uint4 raw[kPieces];
+  float4 L4[GATE == kChannel ? kPieces : 1][2], E4[2];
+  float f[kPieces];
+  const int col = (threadIdx.x % (kTileDim / 8)) * 8, row0 = threadIdx.x / (kTileDim / 8);
+  constexpr int kRowStep = 128 / (kTileDim / 8);
+  const long long channel = static_cast<long long>(h) * p.dim + d0 + col;
+  const bool inside = col < dims;
+  if (GATE == kChannel && inside) {
+    E4[0] = *reinterpret_cast<const float4*>(p.log_decay + last * channels + channel);
+    E4[1] = *reinterpret_cast<const float4*>(p.log_decay + last * channels + channel + 4);
+  }
+#pragma unroll
+  for (int i = 0; i < kPieces; ++i) {
+    const int row = row0 + i * kRowStep;
+    raw[i] = make_uint4(0u, 0u, 0u, 0u);
+    f[i] = 0.0f;
+    if (!inside || row >= c.rows) continue;
+    raw[i] = *reinterpret_cast<const uint4*>(k + row * p.ldk + col);
+    if (GATE == kChannel) {
+      const float* L = p.log_decay + (static_cast<long long>(c.first) + row) * channels + channel;
+      L4[i][0] = *reinterpret_cast<const float4*>(L);
+      L4[i][1] = *reinterpret_cast<const float4*>(L + 4);
+    } else {
+      const long long item = (static_cast<long long>(c.first) + row) * p.heads + h;
+      f[i] = exp_fast(end - p.log_decay[item]) * p.strength[item];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kPieces; ++i) {
+    const int row = row0 + i * kRowStep;
     uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
-    if (row < c.rows && col < dims) {
-      const uint4 raw = *reinterpret_cast<const uint4*>(k + row * p.ldk + col);
-      const uint32_t words[4] = {raw.x, raw.y, raw.z, raw.w};
+    if (inside && row < c.rows) {
+      const uint32_t words[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
       uint32_t a[4], b[4];
       float scale[8];
       if (GATE == kChannel) {
-        const float* L = p.log_decay + (static_cast<long long>(c.first) + row) * channels + static_cast<long long>(h) * p.dim + d0 + col;
-        const float* E = p.log_decay + last * channels + static_cast<long long>(h) * p.dim + d0 + col;
 #pragma unroll
-        for (int i = 0; i < 8; i += 4) {
-          const float4 x = *reinterpret_cast<const float4*>(L + i), y = *reinterpret_cast<const float4*>(E + i);
-          scale[i] = exp_fast(y.x - x.x);
-          scale[i + 1] = exp_fast(y.y - x.y);
-          scale[i + 2] = exp_fast(y.z - x.z);
-          scale[i + 3] = exp_fast(y.w - x.w);
+        for (int j = 0; j < 2; ++j) {
+          scale[4 * j] = exp_fast(E4[j].x - L4[i][j].x);
+          scale[4 * j + 1] = exp_fast(E4[j].y - L4[i][j].y);
+          scale[4 * j + 2] = exp_fast(E4[j].z - L4[i][j].z);
+          scale[4 * j + 3] = exp_fast(E4[j].w - L4[i][j].w);
         }
       } else {
-        const long long item = (static_cast<long long>(c.first) + row) * p.heads + h;
-        const float f = exp_fast(end - p.log_decay[item]) * p.strength[item];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) scale[i] = f;
+        for (int j = 0; j < 8; ++j) scale[j] = f[i];
       }
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float2 x = unpack2(words[i]);
-        const float x0 = x.x * scale[2 * i], x1 = x.y * scale[2 * i + 1];
-        a[i] = mma::pack(x0, x1);
-        b[i] = mma::pack_remainder(x0, x1, a[i]);
+      for (int j = 0; j < 4; ++j) {
+        const float2 x = unpack2(words[j]);
+        const float x0 = x.x * scale[2 * j], x1 = x.y * scale[2 * j + 1];
+        a[j] = mma::pack(x0, x1);
+        b[j] = mma::pack_remainder(x0, x1, a[j]);
       }
       hi = make_uint4(a[0], a[1], a[2], a[3]);
       lo = make_uint4(b[0], b[1], b[2], b[3]);
@@ -515,9 +545,9 @@ memory_chunk_state_kernel(const MemoryArgs p) {
   }
 }
 
-// Block (request, head, 256 pieces of four columns of a row of S); kExp: the key sum is one more piece a row.
+// Block (request, head, 128 pieces of four columns of a row of S); kExp: the key sum is one more piece a row.
 template <int GATE>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(128)
 memory_state_pass_kernel(const MemoryArgs p) {
   __shared__ int first_chunk;
   wait_for_prior_kernels();
@@ -535,7 +565,7 @@ memory_state_pass_kernel(const MemoryArgs p) {
   }
   __syncthreads();
   const int pieces = p.vdim / 4 + (GATE == kExp ? 1 : 0);
-  const int at = blockIdx.z * 256 + threadIdx.x;
+  const int at = blockIdx.z * 128 + threadIdx.x;
   if (at >= p.dim * pieces) return;
   const int d = at / pieces, c4 = at % pieces;
   const bool sums = GATE == kExp && c4 == p.vdim / 4;
@@ -555,27 +585,37 @@ memory_state_pass_kernel(const MemoryArgs p) {
     const long long row = lo + min(n, (c + 1) * kChunkRows) - 1;
     return GATE == kChannel ? p.log_decay[row * p.heads * p.dim + static_cast<long long>(h) * p.dim + d] : p.log_decay[row * p.heads + h];
   };
-  constexpr int kAhead = 8;
-  for (int c0 = 0; c0 < chunks; c0 += kAhead) {
-    float4 u[kAhead];
-    float f[kAhead];
+  constexpr int kAhead = 8;                                  // chunks asked for together, ahead of the ones that are added
+  float4 u[2][kAhead];
+  float f[2][kAhead];
+  auto fetch = [&](int c0, float4 (&uu)[kAhead], float (&ff)[kAhead]) {
 #pragma unroll
     for (int i = 0; i < kAhead; ++i) {
       if (c0 + i >= chunks) continue;
-      f[i] = expf(end_of(c0 + i));
-      if (sums) u[i] = make_float4(U[(c0 + i) * step], 0.0f, 0.0f, 0.0f);
-      else u[i] = *reinterpret_cast<const float4*>(U + (c0 + i) * step);
+      ff[i] = end_of(c0 + i);
+      if (sums) uu[i] = make_float4(U[(c0 + i) * step], 0.0f, 0.0f, 0.0f);
+      else uu[i] = *reinterpret_cast<const float4*>(U + (c0 + i) * step);
     }
+  };
+  auto add = [&](int c0, const float4 (&uu)[kAhead], const float (&ff)[kAhead]) {
 #pragma unroll
     for (int i = 0; i < kAhead; ++i) {
       if (c0 + i >= chunks) continue;
       if (sums) U[(c0 + i) * step] = S.x;
       else *reinterpret_cast<float4*>(U + (c0 + i) * step) = S;
-      S.x = fmaf(f[i], S.x, u[i].x);
-      S.y = fmaf(f[i], S.y, u[i].y);
-      S.z = fmaf(f[i], S.z, u[i].z);
-      S.w = fmaf(f[i], S.w, u[i].w);
+      const float decay = exp_fast(ff[i]);
+      S.x = fmaf(decay, S.x, uu[i].x);
+      S.y = fmaf(decay, S.y, uu[i].y);
+      S.z = fmaf(decay, S.z, uu[i].z);
+      S.w = fmaf(decay, S.w, uu[i].w);
     }
+  };
+  fetch(0, u[0], f[0]);
+  for (int c0 = 0; c0 < chunks; c0 += 2 * kAhead) {
+    fetch(c0 + kAhead, u[1], f[1]);
+    add(c0, u[0], f[0]);
+    fetch(c0 + 2 * kAhead, u[0], f[0]);
+    add(c0 + kAhead, u[1], f[1]);
   }
   if (sums) Sg[0] = S.x;
   else if (wide) *reinterpret_cast<float4*>(Sg) = S;
@@ -651,16 +691,25 @@ memory_chunk_out_kernel(const MemoryArgs p) {
       }
     }
     mma::copy_async_commit();
-    for (int e = tid; e < kTileDim * (VT / 4); e += 128) {
-      const int d = e / (VT / 4), col = (e % (VT / 4)) * 4;
-      uint2 hi = make_uint2(0u, 0u), lo = hi;
-      if (d < dims && col < cols) {
-        const float4 x = *reinterpret_cast<const float4*>(state + static_cast<long long>(d0 + d) * p.ld_state + v0 + col);
-        hi = make_uint2(mma::pack(x.x, x.y), mma::pack(x.z, x.w));
-        lo = make_uint2(mma::pack_remainder(x.x, x.y, hi.x), mma::pack_remainder(x.z, x.w, hi.y));
+    constexpr int kBatch = 8;                                // pieces of the state asked for together
+    static_assert(kTileDim * (VT / 4) % (128 * kBatch) == 0, "whole batches");
+    for (int e0 = tid; e0 < kTileDim * (VT / 4); e0 += 128 * kBatch) {
+      float4 x[kBatch];
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) {
+        const int e = e0 + 128 * i, d = e / (VT / 4), col = (e % (VT / 4)) * 4;
+        x[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (d < dims && col < cols)
+          x[i] = *reinterpret_cast<const float4*>(state + static_cast<long long>(d0 + d) * p.ld_state + v0 + col);
       }
-      *reinterpret_cast<uint2*>(sh + d * (VT + 8) + col) = hi;
-      *reinterpret_cast<uint2*>(sl + d * (VT + 8) + col) = lo;
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) {
+        const int e = e0 + 128 * i, d = e / (VT / 4), col = (e % (VT / 4)) * 4;
+        const uint2 hi = make_uint2(mma::pack(x[i].x, x[i].y), mma::pack(x[i].z, x[i].w));
+        const uint2 lo = make_uint2(mma::pack_remainder(x[i].x, x[i].y, hi.x), mma::pack_remainder(x[i].z, x[i].w, hi.y));
+        *reinterpret_cast<uint2*>(sh + d * (VT + 8) + col) = hi;
+        *reinterpret_cast<uint2*>(sl + d * (VT + 8) + col) = lo;
+      }
     }
     mma::copy_async_wait<0>();
     __syncthreads();
@@ -913,7 +962,7 @@ static int launch_memory_chunks(cudaStream_t s, const MemoryArgs& p, int rows, i
                 state_bytes, s, p);
   PIH_LAUNCH_CHECK();
   const int pieces = p.dim * (p.vdim / 4 + (GATE == kExp ? 1 : 0));
-  launch_kernel(memory_state_pass_kernel<GATE>, dim3(requests, p.heads, (pieces + 255) / 256), dim3(256), 0, s, p);
+  launch_kernel(memory_state_pass_kernel<GATE>, dim3(requests, p.heads, (pieces + 127) / 128), dim3(128), 0, s, p);
   PIH_LAUNCH_CHECK();
   constexpr size_t out_bytes = ChunkOutShape<VT, GATE>::bytes;
   static bool raised = false;                                          // (per instance)
