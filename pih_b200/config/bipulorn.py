@@ -125,7 +125,7 @@ class BipulornConfig:
         sizes = dict(hidden=self.width, heads=_int(m, "heads", where), key_dim=_int(m, "dim", where),
                      value_dim=_int(m, "vdim", where), norm_eps=self.norm_eps)
         if kind == "gla":
-            rank = _int(m, "decay_rank", where) if m.get("decay_rank") is not None else 16
+            rank = _int(m, "decay_rank", where) if m.get("decay_rank") is not None else sizes["key_dim"]
             return GatedLinearSpec(decay_rank=rank, temperature=_number(m, "tau", where), **sizes)
         return MatrixMemorySpec(gate_cap=_number(m, "gate_cap", where), **sizes)
 

@@ -416,7 +416,7 @@ def test_keys_that_stand_out_at_the_windows_edges(dtype, rows_of_step, window, d
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("dim, vdim, rot", [(64, 128, 32), (64, 64, 64), (16, 24, 8), (10, 6, 6), (12, 20, 2), (320, 24, 320), (64, 48, 0)])
+@pytest.mark.parametrize("dim, vdim, rot", [(64, 128, 48), (64, 64, 64), (16, 24, 8), (10, 6, 6), (12, 20, 2), (320, 24, 320), (64, 48, 0)])
 def test_biases_and_rotation_of_neighbouring_pairs(dtype, dim, vdim, rot):
     """q, k and v with their biases added before the rotation, into the queries' buffer and the cache; far positions; pairs of
     halves and of neighbours; rows of padding write nothing."""
